@@ -8,7 +8,8 @@ request rounded up to whole pages), not by slots times the longest sequence.
 
 Layers with the same needs (kv heads, head size, window) form a group with
 storage, block table and free list of its own.  A group with a window gives a
-slot's pages back as soon as every key in them has left the window.
+slot's pages back as soon as every key in them has left the window, the widest one
+where other entries, with windows of their own, read the group's cache.
 
 The reference declares per layer {kv_heads, head_dim, sliding_window, stores,
 source} and keeps one contiguous buffer per storing layer for its single
@@ -85,8 +86,12 @@ class CacheGroup:
     """Storage of the schedule entries that share one CacheRequest."""
 
     def __init__(self, request: CacheRequest, entries: List[int], num_pages: int, num_slots: int,
-                 max_pages_per_slot: int, dtype: torch.dtype, device, stager: Optional[TableStager] = None):
+                 max_pages_per_slot: int, dtype: torch.dtype, device, stager: Optional[TableStager] = None,
+                 reach: Sequence[Tuple[int, int]] = ()):
+        """``reach``: (window, chunk) of every entry that reads this group's cache, its own entries among them (empty:
+        the request's)."""
         self.request = request
+        self.reach = tuple(reach) or ((request.window, request.chunk),)
         self.stager = stager
         self.entries = entries
         self.num_pages = num_pages
@@ -126,15 +131,15 @@ class CacheGroup:
             self.block_table[slot, a:a + need] = torch.tensor(new, dtype=torch.int32)
 
     def trim(self, slot: int, length: int) -> None:
-        """Window and chunk groups: give back the pages whose keys can no longer be read.  The
-        next query sits at position ``length`` and reads keys >= length + 1 - window, and with
+        """Window and chunk groups: give back the pages whose keys can no longer be read by any entry.
+        The next query sits at position ``length`` and reads keys >= length + 1 - window, and with
         chunks none before the start of its own chunk."""
-        chunk = self.request.chunk
-        if not self.window and not chunk:
+        def first(window: int, chunk: int) -> int:
+            lo = max(0, length + 1 - window) if window else 0
+            return max(lo, length - length % chunk) if chunk else lo
+        first_needed = min(first(w, c) for w, c in self.reach)
+        if first_needed < PAGE_TOKENS:
             return
-        first_needed = max(0, length + 1 - self.window) if self.window else 0
-        if chunk:
-            first_needed = max(first_needed, length - length % chunk)
         have = self.slot_pages.get(slot, [])
         back = []
         for lp in range(min(len(have), first_needed // PAGE_TOKENS)):
@@ -173,16 +178,21 @@ class KVCache:
         self.slots = FreeList(self.max_slots, "slot")
         self.lengths: Dict[int, int] = {}
 
-        # groups by request, over the entries that keep a cache of their own
-        by_req: Dict[CacheRequest, List[int]] = {}
+        # groups by request, over the entries that keep a cache of their own, and by how far back their readers look
+        # (an entry that reads another one's cache has a window of its own: the pages stay as long as either needs them)
+        readers: Dict[int, set] = {}
+        for i, (e, r) in enumerate(zip(schedule, requests)):
+            if r is not None:
+                readers.setdefault(i if e.cache_of is None else e.cache_of, set()).add((r.window, r.chunk))
+        by_req: Dict[Tuple, List[int]] = {}
         for i, (e, r) in enumerate(zip(schedule, requests)):
             if r is not None and e.cache_of is None:
-                by_req.setdefault(r, []).append(i)
+                by_req.setdefault((r, tuple(sorted(readers[i]))), []).append(i)
         self.table_stager = TableStager(self.num_pages * max(1, len(by_req)), device)
         self.groups: List[CacheGroup] = [
             CacheGroup(r, ents, self.num_pages, self.max_slots, max_pages_per_slot, dtype, device,
-                       self.table_stager)
-            for r, ents in by_req.items()]
+                       self.table_stager, reach)
+            for (r, reach), ents in by_req.items()]
         where: Dict[int, Tuple[CacheGroup, int]] = {}
         for g in self.groups:
             for j, ent in enumerate(g.entries):
@@ -202,19 +212,7 @@ class KVCache:
                                                    r.num_kv_heads, r.head_dim, r.token_shape, r.dtype, r.value_heads):
                     raise ValueError(f"schedule[{i}] cannot read the cache of entry {src}: different head layout")
                 view = CacheView(pool=g.pool[j], block_table=g.block_table, writes=e.cache_of is None, group=g)
-            st = None
-            if isinstance(s, (tuple, list)):
-                # a mixer made of several (mixers side by side): one tensor per request, None where one asked for nothing
-                made = []
-                for one in s:
-                    made.append(None if one is None else
-                                torch.zeros((self.max_slots, *one.shape), dtype=one.dtype, device=device))
-                    if made[-1] is not None:
-                        self.state_tensors.append(made[-1])
-                st = tuple(made)
-            elif s is not None:
-                st = torch.zeros((self.max_slots, *s.shape), dtype=s.dtype, device=device)
-                self.state_tensors.append(st)
+            st = self._make_state(s)
             self.ios.append(LayerIO(cache=view, state=st))
         # state that the embedding keeps per sequence (``embedding_state``: what it asked for, or None)
         self.embedding_io = LayerIO()
@@ -222,6 +220,17 @@ class KVCache:
             st = torch.zeros((self.max_slots, *embedding_state.shape), dtype=embedding_state.dtype, device=device)
             self.state_tensors.append(st)
             self.embedding_io = LayerIO(state=st)
+
+    def _make_state(self, request):
+        """One tensor [slots, *shape] per request; a tuple of requests (a mixer made of several, a block with state of its
+        own) becomes a tuple, None where one asked for nothing."""
+        if isinstance(request, (tuple, list)):
+            return tuple(self._make_state(one) for one in request)
+        if request is None:
+            return None
+        st = torch.zeros((self.max_slots, *request.shape), dtype=request.dtype, device=self.device)
+        self.state_tensors.append(st)
+        return st
 
     # ---- slots ------------------------------------------------------------------
     def alloc_slot(self) -> int:

@@ -4,6 +4,7 @@ from .nuvilorn import NuvilornConfig
 from .zekazen import ZekazenConfig
 from .lodevik import LodevikConfig
 from .sudupel import SudupelConfig
+from .murilix import MurilixConfig
 
 __all__ = ["ConfigError", "LayerSpec", "ModelSpec", "PartSpec", "ScheduleEntry", "Qwen3Config", "NuvilornConfig",
-           "ZekazenConfig", "LodevikConfig", "SudupelConfig"]
+           "ZekazenConfig", "LodevikConfig", "SudupelConfig", "MurilixConfig"]

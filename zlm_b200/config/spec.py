@@ -44,7 +44,9 @@ class LayerSpec:
     stream, and the norms that go with them.  ``arrangement`` names a registered
     block class (``pre_norm``: h += mixer(norm(h)); h += ffn(norm(h))).  An arrangement with a norm on each
     sublayer's output as well as on its input (``sandwich_norm``) names those in ``mixer_post_norm`` and
-    ``feed_forward_post_norm``."""
+    ``feed_forward_post_norm``.  An arrangement that allows it may pass what the mixer reads through a registered
+    ``mixer_input`` (``causal_conv``), and may end the layer with a ``layer_input`` (``gated_token_input``): something
+    that is added to the stream after the sublayers and reads the step's tokens as well as the stream."""
     arrangement: str
     mixer: PartSpec
     feed_forward: PartSpec
@@ -52,6 +54,8 @@ class LayerSpec:
     feed_forward_norm: PartSpec
     mixer_post_norm: Optional[PartSpec] = None
     feed_forward_post_norm: Optional[PartSpec] = None
+    mixer_input: Optional[PartSpec] = None
+    layer_input: Optional[PartSpec] = None
 
 
 @dataclass(frozen=True)

@@ -1,4 +1,4 @@
-// Embedding gather, RMSNorm over rows of the fp32 residual stream, and SwiGLU.
+// Embedding gather, RMSNorm and LayerNorm over rows of the fp32 residual stream, and SwiGLU.
 // Formulas: src/runtime/executor.zig:714-764 (row lookup, no scale),
 // src/kernels/transformer/norm.zig:4-37 (eps inside the root, x*inv then *w),
 // src/kernels/transformer/activation.zig:8-13 (g / (1 + e^-g) * u).
@@ -244,6 +244,82 @@ extern "C" int zlm_rmsnorm_shares(void* out, int out_dtype, float* x, const void
     else
         ZLM_REQUIRE(false, "rmsnorm_shares: unsupported output dtype %d", out_dtype);
     return zlm_check_launch("rmsnorm_shares");
+}
+
+// ---------------------------------------------------------------- layer norm
+// out[r] = d / sqrt(mean(d^2) + eps) * w with d = x - mean(x): the variance is summed from the deviations, not from the
+// squares.  One block per output row, its size a function of H alone; rows[r] (optional) selects the input row.
+template <typename TO>
+__global__ void layernorm_kernel(TO* __restrict__ out, const float* __restrict__ x, VecW w, const int* __restrict__ rows,
+                                 int H, float eps, int in_regs) {
+    __shared__ float red[32];
+    pdl_trigger();
+    const int r = blockIdx.x;
+    if (rows && !ZLM_CHK(rows + r, 4)) return;
+    const int src = rows ? rows[r] : r;
+    pdl_wait();
+    const float* xr = x + (size_t)src * H;
+    TO* o = out + (size_t)r * H;
+    if (!ZLM_CHK(xr, (size_t)H * 4) || !ZLM_CHK(o, (size_t)H * sizeof(TO)) ||
+        !ZLM_CHK(w.p, (size_t)H * (w.dtype == ZLM_DTYPE_F32 ? 4 : 2)))
+        return;
+    if (in_regs) {
+        const int nv = H / 4;
+        float4 v[NORM_MAX_V4];
+        float s = 0.f;
+#pragma unroll
+        for (int j = 0; j < NORM_MAX_V4; ++j) {
+            const int c = threadIdx.x + j * blockDim.x;
+            v[j] = c < nv ? *(const float4*)(xr + c * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
+            s += (v[j].x + v[j].y) + (v[j].z + v[j].w);
+        }
+        const float mean = block_sum(s, red) / (float)H;
+        float q = 0.f;
+#pragma unroll
+        for (int j = 0; j < NORM_MAX_V4; ++j) {
+            if (threadIdx.x + j * blockDim.x >= nv) continue;
+            v[j].x -= mean; v[j].y -= mean; v[j].z -= mean; v[j].w -= mean;
+            q = fmaf(v[j].x, v[j].x, q); q = fmaf(v[j].y, v[j].y, q); q = fmaf(v[j].z, v[j].z, q); q = fmaf(v[j].w, v[j].w, q);
+        }
+        const float inv = 1.0f / sqrtf(block_sum(q, red) / (float)H + eps);
+#pragma unroll
+        for (int j = 0; j < NORM_MAX_V4; ++j) {
+            const int c = threadIdx.x + j * blockDim.x;
+            if (c >= nv) continue;
+            const float4 wv = w.load4(c * 4);
+            store4(o + c * 4, (v[j].x * inv) * wv.x, (v[j].y * inv) * wv.y, (v[j].z * inv) * wv.z, (v[j].w * inv) * wv.w);
+        }
+        return;
+    }
+    float s = 0.f;
+    for (int i = threadIdx.x; i < H; i += blockDim.x) s += xr[i];
+    const float mean = block_sum(s, red) / (float)H;
+    float q = 0.f;
+    for (int i = threadIdx.x; i < H; i += blockDim.x) {
+        const float d = xr[i] - mean;
+        q = fmaf(d, d, q);
+    }
+    const float inv = 1.0f / sqrtf(block_sum(q, red) / (float)H + eps);
+    for (int i = threadIdx.x; i < H; i += blockDim.x) o[i] = from_f32<TO>(((xr[i] - mean) * inv) * w[i]);
+}
+
+extern "C" int zlm_layernorm(void* out, int out_dtype, const float* x, const void* w, int w_dtype, const int* rows, int R,
+                             int H, float eps, cudaStream_t st) {
+    if (R == 0) return ZLM_OK;
+    ZLM_REQUIRE(R > 0 && H > 0, "layernorm: bad sizes R=%d H=%d", R, H);
+    ZLM_REQUIRE(w_dtype == ZLM_DTYPE_F32 || w_dtype == ZLM_DTYPE_BF16, "layernorm: weight dtype %d", w_dtype);
+    int threads = 128;
+    while (threads < 1024 && threads * 4 * NORM_MAX_V4 < H) threads *= 2;
+    const int in_regs = (H % 4 == 0 && H / 4 <= NORM_MAX_V4 * threads && (uintptr_t)x % 16 == 0 && (uintptr_t)w % 16 == 0 &&
+                         (uintptr_t)out % 16 == 0) ? 1 : 0;
+    const VecW vw{w, w_dtype};
+    if (out_dtype == ZLM_DTYPE_F32)
+        zlm_launch(layernorm_kernel<float>, R, threads, 0, st, (float*)out, x, vw, rows, H, eps, in_regs);
+    else if (out_dtype == ZLM_DTYPE_BF16)
+        zlm_launch(layernorm_kernel<__nv_bfloat16>, R, threads, 0, st, (__nv_bfloat16*)out, x, vw, rows, H, eps, in_regs);
+    else
+        ZLM_REQUIRE(false, "layernorm: unsupported output dtype %d", out_dtype);
+    return zlm_check_launch("layernorm");
 }
 
 // ---------------------------------------------------------------- swiglu

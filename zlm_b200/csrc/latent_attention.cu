@@ -10,6 +10,7 @@
 //   latent_prep          per token: RMSNorm of c with its weight, rotation of kr and of the
 //                        heads' rotated query parts (neighbouring pairs (2i, 2i+1), angle
 //                        pos * inv_freq[i]), the record into the paged pool
+//   latent_down          the same record where queries go through a latent too, which it norms
 //   head_linear          out[t, h, :] = W[h] x[t, h, :] for per-head matrices (folding W_uk
 //                        into the query, W_uv out of the attention's output)
 //   latent_attention     softmax attention of packed query tokens over the paged records;
@@ -18,6 +19,43 @@
 #include "common.cuh"
 
 // ---------------------------------------------------------------------------- prep
+// The record [RMSNorm(src[:r]) * cw | rotated src[r:]] of the token at `pos` of `slot` into its page, and to `row` if
+// given, by the whole block; cosines and sines of the token's angles in shared memory, `red` 32 floats there.
+template <typename TA>
+__device__ __forceinline__ void write_record(const TA* src, const VecW& cw, float eps, const float* cosines, const float* sines,
+                                             int n_rot, int pos, int slot, const int* block_table, int table_stride, TA* pool,
+                                             int dr, int r, TA* row, float* red) {
+    const int ang = n_rot / 2;
+    if (!ZLM_CHK(block_table + (size_t)slot * table_stride + pos / ZLM_PAGE, 4)) return;
+    const int page = block_table[(size_t)slot * table_stride + pos / ZLM_PAGE];
+    TA* rec = pool + ((size_t)page * ZLM_PAGE + pos % ZLM_PAGE) * (r + dr);
+    if (!ZLM_CHK(src, (size_t)(r + dr) * sizeof(TA)) || !ZLM_CHK(rec, (size_t)(r + dr) * sizeof(TA))) return;
+    if (row && !ZLM_CHK(row, (size_t)(r + dr) * sizeof(TA))) return;
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < r; i += blockDim.x) {
+        const float a = to_f32(src[i]);
+        ss = fmaf(a, a, ss);
+    }
+    ss = block_sum(ss, red);
+    const float inv = 1.0f / sqrtf(ss / (float)r + eps);
+    for (int i = threadIdx.x; i < r; i += blockDim.x) {
+        const TA c = from_f32<TA>((to_f32(src[i]) * inv) * cw[i]);
+        rec[i] = c;
+        if (row) row[i] = c;
+    }
+    for (int i = threadIdx.x; i < ang; i += blockDim.x) {
+        const float u = to_f32(src[r + 2 * i]), v = to_f32(src[r + 2 * i + 1]);
+        const TA a = from_f32<TA>(u * cosines[i] - v * sines[i]), b = from_f32<TA>(v * cosines[i] + u * sines[i]);
+        rec[r + 2 * i] = a;
+        rec[r + 2 * i + 1] = b;
+        if (row) { row[r + 2 * i] = a; row[r + 2 * i + 1] = b; }
+    }
+    for (int i = n_rot + threadIdx.x; i < dr; i += blockDim.x) {
+        rec[r + i] = src[r + i];
+        if (row) row[r + i] = src[r + i];
+    }
+}
+
 // One block per token.  q [T, H, dn + dr] and dkv [T, r + dr] are views of the fused projection's rows
 // (dkv is absent for a layer that reads another layer's records).  rec_out (may be null): the token's record also goes
 // to row t of a plain matrix [T, r + dr], for a step that multiplies its own records at once.
@@ -64,37 +102,8 @@ latent_prep_kernel(const TA* q, int q_stride, TA* qo, int qo_stride, int qo_hstr
     }
     if (dkv == nullptr) return;
     if (!ZLM_CHK(token_slot + t, 4)) return;
-    const int slot = token_slot[t];
-    if (!ZLM_CHK(block_table + (size_t)slot * table_stride + pos / ZLM_PAGE, 4)) return;
-    const int page = block_table[(size_t)slot * table_stride + pos / ZLM_PAGE];
-    const TA* src = dkv + (size_t)t * dkv_stride;
-    TA* rec = pool + ((size_t)page * ZLM_PAGE + pos % ZLM_PAGE) * (r + dr);
-    if (!ZLM_CHK(src, (size_t)(r + dr) * sizeof(TA)) || !ZLM_CHK(rec, (size_t)(r + dr) * sizeof(TA))) return;
-    TA* row = rec_out ? rec_out + (size_t)t * rec_stride : nullptr;
-    if (row && !ZLM_CHK(row, (size_t)(r + dr) * sizeof(TA))) return;
-    float ss = 0.f;
-    for (int i = threadIdx.x; i < r; i += blockDim.x) {
-        const float a = to_f32(src[i]);
-        ss = fmaf(a, a, ss);
-    }
-    ss = block_sum(ss, red);
-    const float inv = 1.0f / sqrtf(ss / (float)r + eps);
-    for (int i = threadIdx.x; i < r; i += blockDim.x) {
-        const TA c = from_f32<TA>((to_f32(src[i]) * inv) * cw[i]);
-        rec[i] = c;
-        if (row) row[i] = c;
-    }
-    for (int i = threadIdx.x; i < ang; i += blockDim.x) {
-        const float u = to_f32(src[r + 2 * i]), v = to_f32(src[r + 2 * i + 1]);
-        const TA a = from_f32<TA>(u * cs[0][i] - v * cs[1][i]), b = from_f32<TA>(v * cs[0][i] + u * cs[1][i]);
-        rec[r + 2 * i] = a;
-        rec[r + 2 * i + 1] = b;
-        if (row) { row[r + 2 * i] = a; row[r + 2 * i + 1] = b; }
-    }
-    for (int i = n_rot + threadIdx.x; i < dr; i += blockDim.x) {
-        rec[r + i] = src[r + i];
-        if (row) row[r + i] = src[r + i];
-    }
+    write_record(dkv + (size_t)t * dkv_stride, cw, eps, cs[0], cs[1], n_rot, pos, token_slot[t], block_table, table_stride, pool,
+                 dr, r, rec_out ? rec_out + (size_t)t * rec_stride : nullptr, red);
 }
 
 extern "C" int zlm_latent_prep(const void* q, int q_stride, void* qo, int qo_stride, int qo_hstride, const void* dkv,
@@ -123,6 +132,74 @@ extern "C" int zlm_latent_prep(const void* q, int q_stride, void* qo, int qo_str
     else
         ZLM_REQUIRE(false, "latent_prep: unsupported dtype %d", dtype);
     return zlm_check_launch("latent_prep");
+}
+
+// Queries through a latent of their own: cq[t, :qr] = RMSNorm(down[t, :qr]) * qw (columns of cq from qr up to cq_cols
+// become zeros), and, where the projection has them (dkv not null), the token's record as above.  One block per token.
+template <typename TA>
+__global__ void __launch_bounds__(128)
+latent_down_kernel(TA* __restrict__ cq, int cq_stride, int cq_cols, const TA* __restrict__ down, int down_stride, int qr, VecW qw,
+                   const TA* __restrict__ dkv, VecW cw, float eps, const float* __restrict__ inv_freq, int n_rot,
+                   const int* __restrict__ token_pos, const int* __restrict__ token_slot, const int* __restrict__ block_table,
+                   int table_stride, TA* __restrict__ pool, int dr, int r, TA* __restrict__ rec_out, int rec_stride) {
+    __shared__ float red[32];
+    __shared__ float cs[2][256];
+    pdl_trigger();
+    const int t = blockIdx.x;
+    int pos = 0, slot = 0;
+    if (dkv) {
+        if (!ZLM_CHK(token_pos + t, 4) || !ZLM_CHK(token_slot + t, 4)) return;
+        pos = token_pos[t];
+        slot = token_slot[t];
+        for (int i = threadIdx.x; i < n_rot / 2; i += blockDim.x) {
+            float s, c;
+            sincosf((float)pos * inv_freq[i], &s, &c);
+            cs[0][i] = c;
+            cs[1][i] = s;
+        }
+    }
+    pdl_wait();
+    __syncthreads();
+    const TA* src = down + (size_t)t * down_stride;
+    TA* o = cq + (size_t)t * cq_stride;
+    if (!ZLM_CHK(src, (size_t)qr * sizeof(TA)) || !ZLM_CHK(o, (size_t)cq_cols * sizeof(TA))) return;
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < qr; i += blockDim.x) {
+        const float a = to_f32(src[i]);
+        ss = fmaf(a, a, ss);
+    }
+    ss = block_sum(ss, red);
+    const float inv = 1.0f / sqrtf(ss / (float)qr + eps);
+    for (int i = threadIdx.x; i < cq_cols; i += blockDim.x) o[i] = from_f32<TA>(i < qr ? (to_f32(src[i]) * inv) * qw[i] : 0.f);
+    if (dkv)
+        write_record(dkv + (size_t)t * down_stride, cw, eps, cs[0], cs[1], n_rot, pos, slot, block_table, table_stride, pool, dr, r,
+                     rec_out ? rec_out + (size_t)t * rec_stride : nullptr, red);
+}
+
+extern "C" int zlm_latent_down(void* cq, int cq_stride, int cq_cols, const void* down, int down_stride, int dtype, int qr,
+                               const void* qw, int qw_dtype, const void* dkv, const void* cw, int cw_dtype, float eps,
+                               const float* inv_freq, int n_rot, const int* token_pos, const int* token_slot,
+                               const int* block_table, int table_stride, void* pool, int T, int dr, int r, void* rec_out,
+                               int rec_stride, cudaStream_t st) {
+    if (T == 0) return ZLM_OK;
+    ZLM_REQUIRE(qr > 0 && cq_cols >= qr && cq_stride >= cq_cols && qw, "latent_down: a query latent of %d in rows of %d", qr, cq_cols);
+    ZLM_REQUIRE(dkv || !rec_out, "latent_down: no records to write");
+    if (dkv) {
+        ZLM_REQUIRE(dr >= 0 && r > 0 && pool && block_table && token_slot && token_pos && cw, "latent_down: nowhere to write the records");
+        ZLM_REQUIRE(n_rot >= 0 && n_rot % 2 == 0 && n_rot <= dr && n_rot <= 512 && (n_rot == 0 || inv_freq),
+                    "latent_down: %d rotated dimensions of %d (even, at most 512)", n_rot, dr);
+        ZLM_REQUIRE(!rec_out || rec_stride >= r + dr, "latent_down: the records' second place needs rows of at least %d", r + dr);
+    }
+    const VecW q{qw, qw_dtype}, w{cw ? cw : qw, cw ? cw_dtype : qw_dtype};
+#define ZLM_LD(TA)                                                                                                        \
+    zlm_launch(latent_down_kernel<TA>, T, 128, 0, st, (TA*)cq, cq_stride, cq_cols, (const TA*)down, down_stride, qr, q,       \
+               (const TA*)dkv, w, eps, inv_freq, n_rot, token_pos, token_slot, block_table, table_stride, (TA*)pool, dr, r,  \
+               (TA*)rec_out, rec_stride)
+    if (dtype == ZLM_DTYPE_F32) ZLM_LD(float);
+    else if (dtype == ZLM_DTYPE_BF16) ZLM_LD(__nv_bfloat16);
+    else ZLM_REQUIRE(false, "latent_down: unsupported dtype %d", dtype);
+#undef ZLM_LD
+    return zlm_check_launch("latent_down");
 }
 
 // ---------------------------------------------------------------------------- per-head products

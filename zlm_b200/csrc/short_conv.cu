@@ -13,6 +13,9 @@
 // Heads are padded to `hdp` columns (zeros) in q_out and in the cache, so that keys of `dim` and values of
 // `vdim` columns share the attention kernels' [K|V][kv head][token][hdp] page layout.
 // Sums (taps, squares) are fp32 in both element types.
+//
+// At the end of the file: the same convolution on a whole layer's input, h + conv(h), for designs that convolve what a
+// mixer reads (input_conv).
 #include "common.cuh"
 
 #define SC_WARPS 4
@@ -529,6 +532,86 @@ extern "C" int zlm_norm_gate(void* out, int out_stride, const float* o, const vo
     else
         ZLM_REQUIRE(false, "norm_gate: unsupported dtype %d", dtype);
     return zlm_check_launch("norm_gate");
+}
+
+// ---------------------------------------------------------------------------- a mixer's input convolved
+// out[t] = h[t] + sum_j w[j] * h_(t - taps + 1 + j), per channel, zeros before the sequence's start; w [taps][C].  The
+// rows of earlier steps come from the state, [slots][taps-1][C] in the element type, oldest first (zeros in a new slot).
+// The threads of a sequence's first token of the step do its first taps - 1 tokens, the only ones that read the state,
+// and then bring the state up to date: nobody else touches it.
+template <typename TA, int VEC>
+__global__ void __launch_bounds__(128)
+input_conv_kernel(TA* __restrict__ out, const TA* __restrict__ h, const TA* __restrict__ w, TA* state,
+                  const int* __restrict__ token_seq, const int* __restrict__ cu_seqlens, const int* __restrict__ seq_slot,
+                  int C, int taps) {
+    pdl_trigger();
+    const int t = blockIdx.x, c = (blockIdx.y * blockDim.x + threadIdx.x) * VEC;
+    pdl_wait();
+    if (c >= C || !ZLM_CHK(token_seq + t, 4)) return;
+    const int r = token_seq[t];
+    if (!ZLM_CHK(cu_seqlens + r, 8) || !ZLM_CHK(seq_slot + r, 4)) return;
+    const int row0 = cu_seqlens[r], n = cu_seqlens[r + 1] - row0, i = t - row0;
+    if (i > 0 && i < taps - 1) return;
+    const int last = i == 0 ? max(1, min(n, taps - 1)) : i + 1;
+    TA* st = taps > 1 ? state + (size_t)seq_slot[r] * (taps - 1) * C + c : nullptr;
+    if (i == 0 && st && !ZLM_CHK(st, ((size_t)(taps - 2) * C + VEC) * sizeof(TA))) return;
+    if (!ZLM_CHK(w + c, ((size_t)(taps - 1) * C + VEC) * sizeof(TA))) return;
+    for (int s = i; s < last; ++s) {
+        float a[VEC], u[VEC], k[VEC];
+#pragma unroll
+        for (int v = 0; v < VEC; ++v) a[v] = u[v] = 0.f;
+        for (int j = 0; j < taps; ++j) {
+            const int p = s - (taps - 1) + j;
+            const TA* up = p >= 0 ? h + (size_t)(row0 + p) * C + c : st + (size_t)(taps - 1 + p) * C;
+            if (!ZLM_CHK(up, VEC * sizeof(TA))) continue;
+            load_vec<TA, VEC>(up, u);                   // (the last one is the token's own row)
+            load_vec<TA, VEC>(w + (size_t)j * C + c, k);
+#pragma unroll
+            for (int v = 0; v < VEC; ++v) a[v] = fmaf(k[v], u[v], a[v]);
+        }
+#pragma unroll
+        for (int v = 0; v < VEC; ++v) a[v] += u[v];
+        TA* o = out + (size_t)(row0 + s) * C + c;
+        if (ZLM_CHK(o, VEC * sizeof(TA))) store_vec<TA, VEC>(o, a);
+    }
+    if (i > 0 || taps == 1) return;
+    // the newest taps - 1 rows, in ascending order: a row taken from the old state lies further on than the one written
+    for (int m = 0; m < taps - 1; ++m) {
+        const int p = n - (taps - 1) + m;
+        const TA* up = p >= 0 ? h + (size_t)(row0 + p) * C + c : st + (size_t)(n + m) * C;
+        float u[VEC];
+        if (!ZLM_CHK(up, VEC * sizeof(TA))) continue;
+        load_vec<TA, VEC>(up, u);
+        store_vec<TA, VEC>(st + (size_t)m * C, u);
+    }
+}
+
+template <typename TA>
+static void launch_input_conv(void* out, const void* h, const void* w, void* state, const int* token_seq, const int* cu_seqlens,
+                              const int* seq_slot, int T, int C, int taps, cudaStream_t st) {
+    const size_t quad = 4 * sizeof(TA);
+    const bool vec = C % 4 == 0 && (uintptr_t)out % quad == 0 && (uintptr_t)h % quad == 0 && (uintptr_t)w % quad == 0 &&
+                     (uintptr_t)state % quad == 0;
+    if (vec)
+        zlm_launch(input_conv_kernel<TA, 4>, dim3(T, (C / 4 + 127) / 128), dim3(128), 0, st, (TA*)out, (const TA*)h, (const TA*)w,
+                   (TA*)state, token_seq, cu_seqlens, seq_slot, C, taps);
+    else
+        zlm_launch(input_conv_kernel<TA, 1>, dim3(T, (C + 127) / 128), dim3(128), 0, st, (TA*)out, (const TA*)h, (const TA*)w,
+                   (TA*)state, token_seq, cu_seqlens, seq_slot, C, taps);
+}
+
+extern "C" int zlm_input_conv(void* out, const void* h, const void* w, void* state, int dtype, const int* token_seq,
+                              const int* cu_seqlens, const int* seq_slot, int T, int C, int taps, cudaStream_t st) {
+    if (T == 0) return ZLM_OK;
+    ZLM_REQUIRE(T > 0 && C > 0 && taps >= 1 && (C + 127) / 128 <= 65535, "input_conv: bad sizes T=%d channels=%d taps=%d", T, C, taps);
+    ZLM_REQUIRE(taps == 1 || state, "input_conv: %d taps and no state", taps);
+    if (dtype == ZLM_DTYPE_F32)
+        launch_input_conv<float>(out, h, w, state, token_seq, cu_seqlens, seq_slot, T, C, taps, st);
+    else if (dtype == ZLM_DTYPE_BF16)
+        launch_input_conv<__nv_bfloat16>(out, h, w, state, token_seq, cu_seqlens, seq_slot, T, C, taps, st);
+    else
+        ZLM_REQUIRE(false, "input_conv: unsupported dtype %d", dtype);
+    return zlm_check_launch("input_conv");
 }
 
 ZLM_TRANSLATION_UNIT(short_conv)

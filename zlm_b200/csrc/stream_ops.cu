@@ -4,6 +4,9 @@
 //                    token).  The token before a step's first one is per-slot state.
 //   norm_scale_add   stream[t] += y[t] / sqrt(mean(y[t]^2) + eps) * w (* ls): RMS norm of a sublayer's output, an
 //                    optional second vector (a scale per coordinate of the layer), and the residual add, all in fp32
+//   norm_add_norm    the same (without ls) and the norm, RMS or layer norm, that reads the stream next; in a step of one
+//                    token a sequence also that layer's convolution over time of the normed rows
+//   poly_norm        a polynomial of normed powers as a feed-forward's activation
 //   cast_rows        the stream's rows rounded to the compute dtype (the input of a sublayer that reads the stream
 //                    itself, without a norm before it)
 //   gated_act        out[t, i] = act(gu[t, i]) * gu[t, I + i], act = silu or the tanh form of gelu
@@ -178,12 +181,59 @@ extern "C" int zlm_norm_scale_add(float* stream, const void* y, int y_dtype, con
 }
 
 // ---------------------------------------------------------------- the same, and the norm that reads the stream next
-// stream += y / rms(y) * w1, then out2 = stream / rms(stream) * w2 in the element type: a layer that norms a sublayer's
-// output and the next sublayer's input does both in one pass over the row, which is held in shared memory as fp32.
+// stream += y / rms(y) * w1, then out2 = norm(stream) * w2 in the element type: a layer that norms a sublayer's
+// output and the next sublayer's input does both in one pass over the row, which is held in registers (or, where it does
+// not fit them, in shared memory) as fp32.  norm is x / rms(x), or with CENTER d / rms(d), d = x - mean(x) (layer norm).
 // One block per row, its size a function of H alone.
+//
+// `tail` (steps of one token a sequence; taps 0: none): the next layer's causal convolution over time of the rows just
+// normed, mixed[r] = h + sum_j w[j] * u_j with u the taps - 1 rows before (the slot's state, oldest first) and h itself
+// last; the state then takes h in.  h is the row as out2 holds it.
+struct ConvTail {
+    const void* w;              // [taps][H] in the element type
+    int taps;
+    void* state;                // [slots][taps - 1][H] in the element type
+    const int* seq_slot;
+    void* mixed;                // [rows][H]
+};
 template <typename TO>
+__device__ __forceinline__ float conv_tail_channel(const TO* w, TO* st, int taps, int H, int i, TO hr) {
+    float a = 0.f;
+    for (int j = 0; j < taps - 1; ++j) {
+        const TO u = st[(size_t)j * H + i];
+        a = fmaf(to_f32(w[(size_t)j * H + i]), to_f32(u), a);
+        if (j > 0) st[(size_t)(j - 1) * H + i] = u;
+    }
+    if (taps > 1) st[(size_t)(taps - 2) * H + i] = hr;
+    const float h = to_f32(hr);
+    return h + fmaf(to_f32(w[(size_t)(taps - 1) * H + i]), h, a);
+}
+// the same for four neighbouring channels
+__device__ __forceinline__ float4 tail_load4(const float* p) { return *(const float4*)p; }
+__device__ __forceinline__ float4 tail_load4(const __nv_bfloat16* p) {
+    const uint2 u = *(const uint2*)p;
+    return make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xffff0000u), __uint_as_float(u.y << 16),
+                       __uint_as_float(u.y & 0xffff0000u));
+}
+template <typename TO>
+__device__ __forceinline__ void conv_tail_channels4(const TO* w, TO* st, TO* mixed, int taps, int H, int i, float4 h) {
+    float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int j = 0; j < taps - 1; ++j) {
+        const float4 u = tail_load4(st + (size_t)j * H + i), k = tail_load4(w + (size_t)j * H + i);
+        a.x = fmaf(k.x, u.x, a.x); a.y = fmaf(k.y, u.y, a.y); a.z = fmaf(k.z, u.z, a.z); a.w = fmaf(k.w, u.w, a.w);
+        if (j > 0) store4(st + (size_t)(j - 1) * H + i, u.x, u.y, u.z, u.w);
+    }
+    if (taps > 1) store4(st + (size_t)(taps - 2) * H + i, h.x, h.y, h.z, h.w);
+    const float4 k = tail_load4(w + (size_t)(taps - 1) * H + i);
+    store4(mixed + i, h.x + fmaf(k.x, h.x, a.x), h.y + fmaf(k.y, h.y, a.y), h.z + fmaf(k.z, h.z, a.z), h.w + fmaf(k.w, h.w, a.w));
+}
+template <typename TO> __device__ __forceinline__ float4 as_stored(float4 v) {
+    return make_float4(to_f32(from_f32<TO>(v.x)), to_f32(from_f32<TO>(v.y)), to_f32(from_f32<TO>(v.z)), to_f32(from_f32<TO>(v.w)));
+}
+
+template <typename TO, bool CENTER>
 __global__ void norm_add_norm_kernel(float* __restrict__ stream, const float* __restrict__ y, VecW w1, float eps1,
-                                     TO* __restrict__ out2, VecW w2, float eps2, int H, int in_regs) {
+                                     TO* __restrict__ out2, VecW w2, float eps2, int H, int in_regs, ConvTail tail) {
     extern __shared__ float nan_row[];          // [32] reduction, then (rows that do not fit the registers) [H] the row
     float* red = nan_row;
     float* row = nan_row + 32;
@@ -194,6 +244,16 @@ __global__ void norm_add_norm_kernel(float* __restrict__ stream, const float* __
     const float* yr = y + (size_t)r * H;
     TO* orow = out2 + (size_t)r * H;
     if (!ZLM_CHK(xr, (size_t)H * 4) || !ZLM_CHK(yr, (size_t)H * 4) || !ZLM_CHK(orow, (size_t)H * sizeof(TO))) return;
+    TO *st = nullptr, *mixed = nullptr;
+    const TO* cw = (const TO*)tail.w;
+    if (tail.taps > 0) {
+        if (!ZLM_CHK(tail.seq_slot + r, 4)) return;
+        mixed = (TO*)tail.mixed + (size_t)r * H;
+        if (tail.taps > 1) st = (TO*)tail.state + (size_t)tail.seq_slot[r] * (tail.taps - 1) * H;
+        if (!ZLM_CHK(mixed, (size_t)H * sizeof(TO)) || !ZLM_CHK(cw, (size_t)tail.taps * H * sizeof(TO)) ||
+            (st && !ZLM_CHK(st, (size_t)(tail.taps - 1) * H * sizeof(TO))))
+            return;
+    }
     if (in_regs) {
         // H a multiple of 4 and up to NORM_MAX_V4 float4 a thread: the row is read once and stays in registers
         const int nv = H / 4;
@@ -219,15 +279,33 @@ __global__ void norm_add_norm_kernel(float* __restrict__ stream, const float* __
             a.z += (v[j].z * inv1) * wv.z; a.w += (v[j].w * inv1) * wv.w;
             *(float4*)(xr + c * 4) = a;
             v[j] = a;
-            s2 = fmaf(a.x, a.x, s2); s2 = fmaf(a.y, a.y, s2); s2 = fmaf(a.z, a.z, s2); s2 = fmaf(a.w, a.w, s2);
+            if (CENTER) {
+                s2 += (a.x + a.y) + (a.z + a.w);
+            } else {
+                s2 = fmaf(a.x, a.x, s2); s2 = fmaf(a.y, a.y, s2); s2 = fmaf(a.z, a.z, s2); s2 = fmaf(a.w, a.w, s2);
+            }
         }
-        const float inv2 = 1.0f / sqrtf(block_sum(s2, red) / (float)H + eps2);
+        float sq = block_sum(s2, red);
+        if (CENTER) {
+            const float mean = sq / (float)H;
+            float q = 0.f;
+#pragma unroll
+            for (int j = 0; j < NORM_MAX_V4; ++j) {
+                if (threadIdx.x + j * blockDim.x >= nv) continue;
+                v[j].x -= mean; v[j].y -= mean; v[j].z -= mean; v[j].w -= mean;
+                q = fmaf(v[j].x, v[j].x, q); q = fmaf(v[j].y, v[j].y, q); q = fmaf(v[j].z, v[j].z, q); q = fmaf(v[j].w, v[j].w, q);
+            }
+            sq = block_sum(q, red);
+        }
+        const float inv2 = 1.0f / sqrtf(sq / (float)H + eps2);
 #pragma unroll
         for (int j = 0; j < NORM_MAX_V4; ++j) {
             const int c = threadIdx.x + j * blockDim.x;
             if (c >= nv) continue;
             const float4 wv = w2.load4(c * 4);
-            store4(orow + c * 4, (v[j].x * inv2) * wv.x, (v[j].y * inv2) * wv.y, (v[j].z * inv2) * wv.z, (v[j].w * inv2) * wv.w);
+            const float4 h = make_float4((v[j].x * inv2) * wv.x, (v[j].y * inv2) * wv.y, (v[j].z * inv2) * wv.z, (v[j].w * inv2) * wv.w);
+            store4(orow + c * 4, h.x, h.y, h.z, h.w);
+            if (tail.taps > 0) conv_tail_channels4<TO>(cw, st, mixed, tail.taps, H, c * 4, as_stored<TO>(h));
         }
         return;
     }
@@ -243,30 +321,158 @@ __global__ void norm_add_norm_kernel(float* __restrict__ stream, const float* __
         const float a = xr[i] + (row[i] * inv1) * w1[i];
         xr[i] = a;
         row[i] = a;
-        s2 = fmaf(a, a, s2);
+        s2 = CENTER ? s2 + a : fmaf(a, a, s2);
     }
-    const float inv2 = 1.0f / sqrtf(block_sum(s2, red) / (float)H + eps2);
-    for (int i = threadIdx.x; i < H; i += blockDim.x) orow[i] = from_f32<TO>((row[i] * inv2) * w2[i]);
+    float sq = block_sum(s2, red), mean = 0.f;
+    if (CENTER) {
+        mean = sq / (float)H;
+        float q = 0.f;
+        for (int i = threadIdx.x; i < H; i += blockDim.x) {
+            const float d = row[i] - mean;
+            q = fmaf(d, d, q);
+        }
+        sq = block_sum(q, red);
+    }
+    const float inv2 = 1.0f / sqrtf(sq / (float)H + eps2);
+    for (int i = threadIdx.x; i < H; i += blockDim.x) {
+        const TO h = from_f32<TO>(((row[i] - mean) * inv2) * w2[i]);
+        orow[i] = h;
+        if (tail.taps > 0) mixed[i] = from_f32<TO>(conv_tail_channel<TO>(cw, st, tail.taps, H, i, h));
+    }
 }
 
+template <typename TO>
+static void launch_norm_add_norm(int R, int threads, size_t smem, cudaStream_t st, float* stream, const float* y, VecW v1,
+                                 float eps1, void* out2, VecW v2, float eps2, int H, int in_regs, int center, ConvTail tail) {
+    if (center)
+        zlm_launch(norm_add_norm_kernel<TO, true>, R, threads, smem, st, stream, y, v1, eps1, (TO*)out2, v2, eps2, H, in_regs, tail);
+    else
+        zlm_launch(norm_add_norm_kernel<TO, false>, R, threads, smem, st, stream, y, v1, eps1, (TO*)out2, v2, eps2, H, in_regs, tail);
+}
+
+// center 1: the second norm is a layer norm.  taps 0: no convolution (conv_w, state, seq_slot and mixed are not used).
 extern "C" int zlm_norm_add_norm(float* stream, const float* y, const void* w1, int w1_dtype, float eps1, void* out2,
-                                 int out2_dtype, const void* w2, int w2_dtype, float eps2, int R, int H, cudaStream_t st) {
+                                 int out2_dtype, const void* w2, int w2_dtype, float eps2, int R, int H, int center,
+                                 const void* conv_w, int taps, void* state, const int* seq_slot, void* mixed, cudaStream_t st) {
     if (R == 0) return ZLM_OK;
     ZLM_REQUIRE(R > 0 && H > 0 && H <= 11264, "norm_add_norm: bad sizes R=%d H=%d (rows of up to 11264)", R, H);
+    ZLM_REQUIRE(taps >= 0 && (taps == 0 || (conv_w && mixed && seq_slot && (taps == 1 || state))),
+                "norm_add_norm: a convolution of %d taps needs its weights, the slots' state and a place for its rows", taps);
     int threads = 128;
     while (threads < 1024 && threads * 4 * NORM_MAX_V4 < H) threads *= 2;
     const int in_regs = (H % 4 == 0 && H / 4 <= NORM_MAX_V4 * threads && (uintptr_t)stream % 16 == 0 && (uintptr_t)y % 16 == 0 &&
-                         (uintptr_t)w1 % 16 == 0 && (uintptr_t)w2 % 16 == 0 && (uintptr_t)out2 % 16 == 0) ? 1 : 0;
+                         (uintptr_t)w1 % 16 == 0 && (uintptr_t)w2 % 16 == 0 && (uintptr_t)out2 % 16 == 0 &&
+                         (uintptr_t)conv_w % 16 == 0 && (uintptr_t)state % 16 == 0 && (uintptr_t)mixed % 16 == 0) ? 1 : 0;
     const size_t smem = (size_t)(32 + (in_regs ? 0 : H)) * sizeof(float);
     const VecW v1{w1, w1_dtype}, v2{w2, w2_dtype};
+    const ConvTail tail{conv_w, taps, state, seq_slot, mixed};
     if (out2_dtype == ZLM_DTYPE_F32)
-        zlm_launch(norm_add_norm_kernel<float>, R, threads, smem, st, stream, y, v1, eps1, (float*)out2, v2, eps2, H, in_regs);
+        launch_norm_add_norm<float>(R, threads, smem, st, stream, y, v1, eps1, out2, v2, eps2, H, in_regs, center, tail);
     else if (out2_dtype == ZLM_DTYPE_BF16)
-        zlm_launch(norm_add_norm_kernel<__nv_bfloat16>, R, threads, smem, st, stream, y, v1, eps1, (__nv_bfloat16*)out2, v2,
-                   eps2, H, in_regs);
+        launch_norm_add_norm<__nv_bfloat16>(R, threads, smem, st, stream, y, v1, eps1, out2, v2, eps2, H, in_regs, center, tail);
     else
         ZLM_REQUIRE(false, "norm_add_norm: unsupported output dtype %d", out2_dtype);
     return zlm_check_launch("norm_add_norm");
+}
+
+// ---------------------------------------------------------------- a polynomial of normed powers
+// out[t] = a N(z) + b N(z^2) + c N(z^3) + e over the row z[t] of ff values (powers element by element, N(u) = u /
+// sqrt(mean(u^2) + eps)), the four numbers in `coef`; columns of out from ff up to out_cols become zeros.  Sums and
+// norms fp32.  One block per row, its size a function of ff alone.
+#define PN_MAX_V 4
+template <typename TA> struct PolyVec;          // eight neighbouring elements
+template <> struct PolyVec<__nv_bfloat16> {
+    uint4 u;
+    __device__ __forceinline__ void load(const __nv_bfloat16* p) { u = *(const uint4*)p; }
+    __device__ __forceinline__ float get(int i) const {
+        const unsigned w = i < 2 ? u.x : (i < 4 ? u.y : (i < 6 ? u.z : u.w));
+        return __uint_as_float((i & 1) ? (w & 0xffff0000u) : (w << 16));
+    }
+};
+template <> struct PolyVec<float> {
+    float4 a, b;
+    __device__ __forceinline__ void load(const float* p) { a = *(const float4*)p; b = *(const float4*)(p + 4); }
+    __device__ __forceinline__ float get(int i) const {
+        const float4 v = i < 4 ? a : b;
+        const int k = i & 3;
+        return k == 0 ? v.x : (k == 1 ? v.y : (k == 2 ? v.z : v.w));
+    }
+};
+template <typename TA>
+__global__ void poly_norm_kernel(TA* __restrict__ out, int out_stride, int out_cols, const TA* __restrict__ z, int z_stride,
+                                 VecW coef, int F, float eps, int in_regs) {
+    __shared__ float red[32];
+    pdl_trigger();
+    const int t = blockIdx.x;
+    pdl_wait();
+    const TA* zr = z + (size_t)t * z_stride;
+    TA* o = out + (size_t)t * out_stride;
+    if (!ZLM_CHK(zr, (size_t)F * sizeof(TA)) || !ZLM_CHK(o, (size_t)out_cols * sizeof(TA)) ||
+        !ZLM_CHK(coef.p, 4 * (coef.dtype == ZLM_DTYPE_F32 ? 4 : 2)))
+        return;
+    float s1 = 0.f, s2 = 0.f, s3 = 0.f;
+    auto add = [&](float v) {
+        const float q = v * v;
+        s1 += q;
+        s2 = fmaf(q, q, s2);
+        s3 = fmaf(q * q, q, s3);
+    };
+    PolyVec<TA> keep[PN_MAX_V];
+    const int nv = F / 8;
+    if (in_regs) {
+#pragma unroll
+        for (int j = 0; j < PN_MAX_V; ++j) {
+            const int c = threadIdx.x + j * blockDim.x;
+            if (c < nv) keep[j].load(zr + c * 8);
+        }
+#pragma unroll
+        for (int j = 0; j < PN_MAX_V; ++j) {
+            if (threadIdx.x + j * blockDim.x >= nv) continue;
+#pragma unroll
+            for (int i = 0; i < 8; ++i) add(keep[j].get(i));
+        }
+    } else {
+        for (int i = threadIdx.x; i < F; i += blockDim.x) add(to_f32(zr[i]));
+    }
+    const float f = (float)F;
+    const float ka = coef[0] / sqrtf(block_sum(s1, red) / f + eps);
+    const float kb = coef[1] / sqrtf(block_sum(s2, red) / f + eps);
+    const float kc = coef[2] / sqrtf(block_sum(s3, red) / f + eps);
+    const float ke = coef[3];
+    auto value = [&](float v) { return fmaf(v, fmaf(v, fmaf(v, kc, kb), ka), ke); };
+    if (in_regs) {
+#pragma unroll
+        for (int j = 0; j < PN_MAX_V; ++j) {
+            const int c = threadIdx.x + j * blockDim.x;
+            if (c >= nv) continue;
+            store4(o + c * 8, value(keep[j].get(0)), value(keep[j].get(1)), value(keep[j].get(2)), value(keep[j].get(3)));
+            store4(o + c * 8 + 4, value(keep[j].get(4)), value(keep[j].get(5)), value(keep[j].get(6)), value(keep[j].get(7)));
+        }
+    } else {
+        for (int i = threadIdx.x; i < F; i += blockDim.x) o[i] = from_f32<TA>(value(to_f32(zr[i])));
+    }
+    for (int i = F + threadIdx.x; i < out_cols; i += blockDim.x) o[i] = from_f32<TA>(0.f);
+}
+
+extern "C" int zlm_poly_norm(void* out, int out_stride, int out_cols, const void* z, int z_stride, int dtype, const void* coef,
+                             int coef_dtype, int T, int F, float eps, cudaStream_t st) {
+    if (T == 0) return ZLM_OK;
+    ZLM_REQUIRE(T > 0 && F > 0 && out_cols >= F && out_stride >= out_cols && z_stride >= F, "poly_norm: bad sizes T=%d F=%d", T, F);
+    int threads = 128;
+    while (threads < 1024 && threads * 8 * PN_MAX_V < F) threads *= 2;
+    const int el = dtype == ZLM_DTYPE_F32 ? 4 : 2;
+    const int in_regs = (F % 8 == 0 && F <= threads * 8 * PN_MAX_V && ((size_t)z_stride * el) % 16 == 0 &&
+                         ((size_t)out_stride * el) % 16 == 0 && (uintptr_t)z % 16 == 0 && (uintptr_t)out % 16 == 0) ? 1 : 0;
+    const VecW c{coef, coef_dtype};
+    if (dtype == ZLM_DTYPE_F32)
+        zlm_launch(poly_norm_kernel<float>, T, threads, 0, st, (float*)out, out_stride, out_cols, (const float*)z, z_stride, c, F,
+                   eps, in_regs);
+    else if (dtype == ZLM_DTYPE_BF16)
+        zlm_launch(poly_norm_kernel<__nv_bfloat16>, T, threads, 0, st, (__nv_bfloat16*)out, out_stride, out_cols,
+                   (const __nv_bfloat16*)z, z_stride, c, F, eps, in_regs);
+    else
+        ZLM_REQUIRE(false, "poly_norm: unsupported dtype %d", dtype);
+    return zlm_check_launch("poly_norm");
 }
 
 // ---------------------------------------------------------------- the stream's rows in the compute dtype

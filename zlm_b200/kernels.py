@@ -34,6 +34,15 @@ def interleave_gate_up(gate: torch.Tensor, up: torch.Tensor) -> torch.Tensor:
     return torch.stack([gate.view(I // 8, 8, K), up.view(I // 8, 8, K)], dim=1).reshape(2 * I, K).contiguous()
 
 
+def pad_inner(w: torch.Tensor) -> torch.Tensor:
+    """``w`` [N, K] with columns of zeros up to a multiple of 8 in bfloat16 (the products read 16 bytes of a row at a
+    time); the activations that meet it are then padded with zeros as well."""
+    extra = -w.shape[1] % 8
+    if w.dtype != torch.bfloat16 or not extra:
+        return w
+    return torch.nn.functional.pad(w, (0, extra)).contiguous()
+
+
 def attention_len_bucket(max_len: int) -> int:
     """The longest sequence of a step in pages, rounded up: powers of two up to 8, then
     multiples of 8.  The decode attention sizes its grid by it, so a captured decode step
@@ -369,6 +378,16 @@ class CudaKernels:
         self._call("zlm_rmsnorm", self._p(out), c_int(_dt(out)), self._p(x),
                    self._p(w), c_int(_dt(w)), self._p(rows), c_int(R), c_int(H),
                    c_float(eps), self._stream())
+
+    def layernorm(self, out: torch.Tensor, x: torch.Tensor, w: torch.Tensor, eps: float,
+                  rows: Optional[torch.Tensor] = None) -> None:
+        """out[r] = d / sqrt(mean(d^2) + eps) * w with d = x[rows[r] or r] - its mean; x is the fp32 stream."""
+        R, H = out.shape
+        assert x.dtype == torch.float32 and x.shape[1] == H and w.shape == (H,)
+        assert out.is_contiguous() and x.is_contiguous() and w.is_contiguous()
+        assert rows is None or (rows.dtype == torch.int32 and rows.numel() >= R)
+        self._call("zlm_layernorm", self._p(out), c_int(_dt(out)), self._p(x), self._p(w), c_int(_dt(w)), self._p(rows),
+                   c_int(R), c_int(H), c_float(eps), self._stream())
 
     def swiglu(self, out: torch.Tensor, gu: torch.Tensor) -> None:
         """out[t, i] = silu(gu[t, i]) * gu[t, I + i]."""
@@ -937,6 +956,30 @@ class CudaKernels:
                            c_int(T), c_int(N), c_int(K), c_int(ldx), c_int(ldy), c_int(STORE_F32), ps, st)
         call(2)
 
+    def mingru(self, out: torch.Tensor, proj: torch.Tensor, z_off: int, x_off: int, g_off: int, bz: Optional[torch.Tensor],
+               bx: Optional[torch.Tensor], state: torch.Tensor, plan, pieces: Optional[bool] = None) -> None:
+        """out[t] = S_t silu(g), S_t = (1 - z) S_(t-1) + z cand, z = sigmoid(zp + bz), cand = u + 1/2 where u = xp + bx >= 0
+        and sigmoid(u) elsewhere; zp, xp and g are the W columns of ``proj`` from z_off, x_off and g_off on, ``state``
+        [slots, W] fp32.  Long prompts run in pieces side by side (``pieces`` forces or forbids that)."""
+        T = proj.shape[0]
+        W = state.shape[1]
+        assert out.shape == (T, W) and out.dtype == proj.dtype and out.stride(1) == 1 and proj.stride(1) == 1
+        assert state.dtype == torch.float32 and state.dim() == 2 and state.is_contiguous()
+        for b in (bz, bx):
+            assert b is None or (b.shape == (W,) and b.is_contiguous() and b.dtype == (bz if bz is not None else bx).dtype)
+        max_new = int(getattr(plan, "max_new", 0) or 0)
+        if pieces is None:
+            pieces = max_new >= self.RECURRENT_PIECES_FROM
+        part = None
+        if pieces:
+            maxp = (max_new + self.RECURRENT_PIECE - 1) // self.RECURRENT_PIECE
+            part = plan.scratch("mingru.pieces", (2 * plan.R * maxp * W,), torch.float32)
+        b = bz if bz is not None else bx
+        self._call("zlm_mingru", self._p(out), c_int(out.stride(0)), self._p(proj), c_int(proj.stride(0)), c_int(z_off),
+                   c_int(x_off), c_int(g_off), self._p(bz), self._p(bx), c_int(_dt(b) if b is not None else F32), self._p(state),
+                   c_int(_dt(proj)), self._p(plan.seq_slot), self._p(plan.cu_seqlens), c_int(T), c_int(plan.R), c_int(W),
+                   c_int(max_new), self._p(part), self._stream())
+
     def lowrank_decay(self, alpha: torch.Tensor, proj: torch.Tensor, lo_off: int, w2: torch.Tensor, b: Optional[torch.Tensor],
                       tau: float) -> None:
         """alpha [T, C] fp32 = sigmoid(w2 lo + b)^(1/tau), lo = ``rank`` columns of proj from lo_off on, w2 [C, rank]."""
@@ -1041,6 +1084,37 @@ class CudaKernels:
                    c_int(block_table.stride(0) if dkv is not None else 0), self._p(pool if dkv is not None else None),
                    c_int(T), c_int(heads), c_int(dim), c_int(rot_dim), c_int(kv_rank), self._p(rec_out),
                    c_int(rec_out.stride(0) if rec_out is not None else 0), self._stream())
+
+    def latent_down(self, cq: torch.Tensor, down: torch.Tensor, q_weight: torch.Tensor, eps: float,
+                    dkv: Optional[torch.Tensor] = None, c_weight: Optional[torch.Tensor] = None,
+                    inv_freq: Optional[torch.Tensor] = None, n_rot: int = 0, token_pos: Optional[torch.Tensor] = None,
+                    token_slot: Optional[torch.Tensor] = None, block_table: Optional[torch.Tensor] = None,
+                    pool: Optional[torch.Tensor] = None, rot_dim: int = 0, kv_rank: int = 0,
+                    rec_out: Optional[torch.Tensor] = None) -> None:
+        """cq[t] = RMSNorm(down[t]) * q_weight (``down`` [T, q_rank], columns of cq beyond q_rank become zeros); with ``dkv``
+        also the token's record, as ``latent_prep`` writes it (``down`` and ``dkv`` are column views of one projection)."""
+        T, qr = down.shape
+        assert cq.shape[0] == T and cq.shape[1] >= qr and cq.dtype == down.dtype and cq.stride(1) == 1 and down.stride(1) == 1
+        assert q_weight.shape == (qr,) and q_weight.is_contiguous()
+        if inv_freq is not None and n_rot:
+            assert inv_freq.dtype == torch.float32 and inv_freq.numel() * 2 == n_rot
+        else:
+            inv_freq, n_rot = None, 0
+        if dkv is not None:
+            assert dkv.shape == (T, kv_rank + rot_dim) and dkv.stride() == down.stride() and dkv.dtype == down.dtype
+            assert pool is not None and pool.dtype == down.dtype and pool.is_contiguous()
+            assert tuple(pool.shape[1:]) == (PAGE_TOKENS, kv_rank + rot_dim) and block_table.dtype == torch.int32
+            assert c_weight is not None and c_weight.shape == (kv_rank,) and c_weight.is_contiguous()
+        else:
+            inv_freq = block_table = pool = c_weight = token_pos = token_slot = None
+        assert rec_out is None or (dkv is not None and rec_out.shape == (T, kv_rank + rot_dim) and rec_out.stride(1) == 1
+                                   and rec_out.dtype == down.dtype)
+        self._call("zlm_latent_down", self._p(cq), c_int(cq.stride(0)), c_int(cq.shape[1]), self._p(down), c_int(down.stride(0)),
+                   c_int(_dt(down)), c_int(qr), self._p(q_weight), c_int(_dt(q_weight)), self._p(dkv), self._p(c_weight),
+                   c_int(_dt(c_weight) if c_weight is not None else F32), c_float(eps), self._p(inv_freq), c_int(n_rot),
+                   self._p(token_pos), self._p(token_slot), self._p(block_table),
+                   c_int(block_table.stride(0) if block_table is not None else 0), self._p(pool), c_int(T), c_int(rot_dim),
+                   c_int(kv_rank), self._p(rec_out), c_int(rec_out.stride(0) if rec_out is not None else 0), self._stream())
 
     def latent_gather(self, rec: torch.Tensor, pool: torch.Tensor, block_table: torch.Tensor, token_pos: torch.Tensor,
                       token_slot: torch.Tensor) -> None:
@@ -1173,17 +1247,79 @@ class CudaKernels:
     NORM_ADD_NORM_MAX = 11264        # the widest row the fused pair of norms holds in shared memory
 
     def norm_add_norm(self, stream: torch.Tensor, y: torch.Tensor, w1: torch.Tensor, eps1: float, out2: torch.Tensor,
-                      w2: torch.Tensor, eps2: float) -> None:
+                      w2: torch.Tensor, eps2: float, center: bool = False, conv=None) -> None:
         """stream[t] += y[t] / sqrt(mean(y[t]^2) + eps1) * w1, then out2[t] = stream[t] / sqrt(mean(stream[t]^2) + eps2)
         * w2 (the compute dtype): a sublayer's closing norm with its residual add, and the next sublayer's opening norm,
-        in one kernel.  y fp32."""
+        in one kernel.  y fp32.  ``center``: the opening norm is a layer norm (the mean taken off first).  ``conv``
+        (a step of one token a sequence): (mixed, taps [taps, H], state [slots, taps-1, H], plan), for
+        ``input_conv(mixed, out2, taps, state, plan)`` in the same kernel."""
         R, H = stream.shape
         assert stream.dtype == y.dtype == torch.float32 and y.shape == (R, H) and out2.shape == (R, H)
         assert stream.is_contiguous() and y.is_contiguous() and out2.is_contiguous() and H <= self.NORM_ADD_NORM_MAX
         assert w1.shape == (H,) and w2.shape == (H,) and w1.is_contiguous() and w2.is_contiguous()
+        mixed = cw = state = slots = None
+        taps = 0
+        if conv is not None:
+            mixed, cw, state, plan = conv
+            taps, slots = self._check_input_conv(mixed, out2, cw, state), plan.seq_slot
+            assert plan.is_decode and plan.R == R
         self._call("zlm_norm_add_norm", self._p(stream), self._p(y), self._p(w1), c_int(_dt(w1)), c_float(eps1),
                    self._p(out2), c_int(_dt(out2)), self._p(w2), c_int(_dt(w2)), c_float(eps2), c_int(R), c_int(H),
+                   c_int(1 if center else 0), self._p(cw), c_int(taps), self._p(state if taps > 1 else None), self._p(slots),
+                   self._p(mixed), self._stream())
+
+    @staticmethod
+    def _check_input_conv(out, h, w, state) -> int:
+        taps, C = w.shape
+        assert h.shape[1] == C and out.shape == h.shape and out.dtype == h.dtype == w.dtype
+        assert out.is_contiguous() and h.is_contiguous() and w.is_contiguous()
+        if taps > 1:
+            assert state is not None and tuple(state.shape[1:]) == (taps - 1, C) and state.dtype == h.dtype and state.is_contiguous()
+        return taps
+
+    def input_conv(self, out: torch.Tensor, h: torch.Tensor, w: torch.Tensor, state: Optional[torch.Tensor], plan) -> None:
+        """out[t] = h[t] + sum_j w[j] * h_(t - taps + 1 + j), channel by channel over the tokens of a sequence, zeros
+        before its start; w [taps, C].  The rows before a step's first token come from ``state`` [slots, taps-1, C], oldest
+        first, which is brought up to date."""
+        taps = self._check_input_conv(out, h, w, state)
+        T, C = h.shape
+        self._call("zlm_input_conv", self._p(out), self._p(h), self._p(w), self._p(state if taps > 1 else None), c_int(_dt(h)),
+                   self._p(plan.token_seq), self._p(plan.cu_seqlens), self._p(plan.seq_slot), c_int(T), c_int(C), c_int(taps),
                    self._stream())
+
+    def poly_norm(self, out: torch.Tensor, z: torch.Tensor, coef: torch.Tensor, eps: float) -> None:
+        """out[t] = a N(z[t]) + b N(z[t]^2) + c N(z[t]^3) + e, powers element by element, N(u) = u / sqrt(mean(u^2) + eps)
+        over the row, (a, b, c, e) = ``coef`` [4]; columns of ``out`` beyond z's become zeros."""
+        T, F = z.shape
+        assert out.shape[0] == T and out.shape[1] >= F and out.dtype == z.dtype and out.stride(1) == 1 and z.stride(1) == 1
+        assert coef.shape == (4,) and coef.is_contiguous()
+        self._call("zlm_poly_norm", self._p(out), c_int(out.stride(0)), c_int(out.shape[1]), self._p(z), c_int(z.stride(0)),
+                   c_int(_dt(z)), self._p(coef), c_int(_dt(coef)), c_int(T), c_int(F), c_float(eps), self._stream())
+
+    # -- a layer's second look at its tokens (see csrc/token_input.cu) -------------------------------------------
+    def token_gate(self, g: torch.Tensor, z: torch.Tensor, side: torch.Tensor, off: int, ids: torch.Tensor) -> None:
+        """g[t] = gelu_tanh(z[t]) * side[ids[t], off : off + dim], dim = z's columns; columns of g beyond them become zeros."""
+        T, dim = z.shape
+        assert g.shape[0] == T and g.shape[1] >= dim and g.dtype == z.dtype == side.dtype and ids.dtype == torch.int32
+        assert g.stride(1) == 1 and z.stride(1) == 1 and side.is_contiguous() and 0 <= off and off + dim <= side.shape[1]
+        self._call("zlm_token_gate", self._p(g), c_int(g.stride(0)), c_int(g.shape[1]), self._p(z), c_int(z.stride(0)),
+                   self._p(side), c_int(side.shape[1]), c_int(off), self._p(ids), c_int(_dt(z)), c_int(T), c_int(dim),
+                   c_int(side.shape[0]), self._stream())
+
+    def token_gate_few_supported(self, tokens: int, w: torch.Tensor) -> bool:
+        return w.dtype == torch.bfloat16 and bool(self.lib.zlm_token_gate_few_supported(c_int(tokens), c_int(w.shape[1])))
+
+    def token_gate_few(self, g: torch.Tensor, x: torch.Tensor, w: torch.Tensor, side: torch.Tensor, off: int,
+                       ids: torch.Tensor) -> None:
+        """``token_gate`` with z = x w^T in the same kernel, for up to 16 tokens: x the fp32 stream [T, K], w [dim, K] bf16."""
+        T, K = x.shape
+        dim = w.shape[0]
+        assert x.dtype == torch.float32 and x.is_contiguous() and w.shape == (dim, K) and w.is_contiguous()
+        assert g.shape[0] == T and g.shape[1] >= dim and g.dtype == w.dtype == side.dtype == torch.bfloat16
+        assert g.stride(1) == 1 and side.is_contiguous() and 0 <= off and off + dim <= side.shape[1] and ids.dtype == torch.int32
+        self._call("zlm_token_gate_few", self._p(g), c_int(g.stride(0)), c_int(g.shape[1]), self._p(x), self._p(w),
+                   self._p(side), c_int(side.shape[1]), c_int(off), self._p(ids), c_int(T), c_int(K), c_int(dim),
+                   c_int(side.shape[0]), self._stream())
 
     def cast_rows(self, out: torch.Tensor, x: torch.Tensor) -> None:
         """out = x rounded to bfloat16 (x fp32, both contiguous and of one shape)."""

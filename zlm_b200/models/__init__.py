@@ -4,3 +4,4 @@ from . import nuvilorn   # noqa: F401
 from . import zekazen   # noqa: F401
 from . import lodevik   # noqa: F401
 from . import sudupel   # noqa: F401
+from . import murilix   # noqa: F401

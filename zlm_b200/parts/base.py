@@ -133,7 +133,7 @@ class CacheView:
 class LayerIO:
     """What one schedule entry owns beside its weights."""
     cache: Optional[CacheView] = None
-    state: Any = None     # [slots, *StateRequest.shape]; a tuple of such tensors where the mixer asked with a tuple of requests
+    state: Any = None     # [slots, *StateRequest.shape]; a tuple of such (or None) where the mixer, or its block, asked with a tuple of requests
 
 
 @dataclass

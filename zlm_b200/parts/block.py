@@ -10,6 +10,10 @@ sublayers read the stream itself.  The norm may carry a scale per coordinate of 
 
 ``sandwich_norm``: h = h + post1(mixer(pre1(h))); h = h + post2(ffn(pre2(h))): a norm on what a sublayer reads and
 another on what it gives.
+
+``parallel_sublayers``: with n = norm(h), h = h + (mixer(n) + ffn(n)): one norm, both sublayers read its rows.  What the
+mixer reads may pass through a mixer input first (a convolution over time), and a layer input may follow the sublayers
+(something read from the step's tokens and added to the stream behind a norm of its own).
 """
 from __future__ import annotations
 
@@ -19,6 +23,7 @@ import torch
 
 from ..registry import register_arrangement
 from .base import FeedForward, LayerIO, Mixer, Norm, Part, StepContext
+from .norm import NoNorm
 
 
 @register_arrangement("pre_norm")
@@ -210,3 +215,93 @@ class SandwichNormBlock(Part):
                        lambda x, y: self.mixer.forward(x, y, ctx, io), ctx)
         if has_ffn:
             self._sublayer(self.ffn_norm, self.ffn_post, after, hidden, lambda x, y: self.ffn.forward(x, y, ctx), ctx)
+
+
+@register_arrangement("parallel_sublayers")
+class ParallelSublayersBlock(Part):
+    """x <- x + (mixer(m) + ffn(n)) with n = norm(x) and m = n, or what ``mixer_input`` makes of n; then ``layer_input``.
+
+    Both sublayers add their results into the stream themselves.  A layer input ends with a norm whose result is added to
+    the stream; where a block of this arrangement follows, that kernel also leaves the next block's n and, in steps of one
+    token a sequence, its m.  ``LayerIO.state`` is (the mixer's state, the mixer input's state) if either has any."""
+
+    def __init__(self, hidden_size: int, mixer: Mixer, feed_forward: FeedForward, mixer_norm: Norm, feed_forward_norm: Norm,
+                 mixer_input: Optional[Part] = None, layer_input: Optional[Part] = None):
+        self.hidden = int(hidden_size)
+        self.mixer, self.ffn = mixer, feed_forward
+        self.norm = mixer_norm                   # (the feed-forward has no norm of its own)
+        self.mixer_input, self.layer_input = mixer_input, layer_input
+        if not isinstance(feed_forward_norm, NoNorm):
+            raise ValueError("parallel_sublayers: the sublayers share one norm; feed_forward_norm must be 'none'")
+
+    def children(self) -> Dict[str, Part]:
+        c = {"mixer": self.mixer, "feed_forward": self.ffn, "mixer_norm": self.norm}
+        for name in ("mixer_input", "layer_input"):
+            if getattr(self, name) is not None:
+                c[name] = getattr(self, name)
+        return c
+
+    graph_safe = PreNormBlock.graph_safe
+    prefers_plain_launches = PreNormBlock.prefers_plain_launches
+    step_key = PreNormBlock.step_key
+
+    def state_request(self):
+        asks = (self.mixer.state_request(), self.mixer_input.state_request() if self.mixer_input is not None else None)
+        return asks if any(a is not None for a in asks) else None
+
+    def first_norm_weight(self):
+        return None             # (no product prepares this block's norm: see ``first_norm``)
+
+    def first_norm(self) -> Norm:
+        return self.norm
+
+    @staticmethod
+    def _states(io: LayerIO):
+        return io.state if isinstance(io.state, tuple) else (None, None)
+
+    def forward(self, hidden: torch.Tensor, ctx: StepContext, io: LayerIO) -> None:
+        rt, k = self.rt, self.rt.k
+        self.finish_products()          # (a block of another arrangement before this one may have left its last product)
+        ctx.extras.pop("stream.rounded", None)
+        for word in ("expect_norm", "norm_output_read_by_products"):
+            say = getattr(k, word, None)
+            if say is not None:
+                say(None if word == "expect_norm" else False)
+        mixer_state, input_state = self._states(io)
+        n = rt.ws.get("block.normed", hidden.shape, rt.dtype)
+        mixed_by = ctx.extras.pop("stream.mixed", None)
+        # (what closed the block before may have left this block's normed rows, and the mixer's, there)
+        if ctx.extras.pop("stream.normed", None) != (n.data_ptr(), id(self.norm)):
+            self.norm.forward(n, hidden)
+            mixed_by = None
+        m = n
+        if self.mixer_input is not None:
+            m = rt.ws.get("block.mixed", hidden.shape, rt.dtype)
+            if mixed_by != (m.data_ptr(), id(self.mixer_input)):
+                self.mixer_input.forward(m, n, ctx, input_state)
+        self.mixer.forward(m, hidden, ctx, LayerIO(cache=io.cache, state=mixer_state))
+        if not getattr(self.ffn, "is_identity", False):
+            self.ffn.forward(n, hidden, ctx)
+        if self.layer_input is not None:
+            self._close(hidden, ctx, n)
+
+    def _close(self, hidden: torch.Tensor, ctx: StepContext, n: torch.Tensor) -> None:
+        """The layer input, and with its closing norm the next block's opening one (the model's word on who follows)."""
+        y = self.layer_input.project(hidden, ctx)
+        post = self.layer_input.norm
+        fuse = getattr(post, "add_into_then_norm", None)
+        nxt = ctx.extras.get("first_norm_after_block")
+        if nxt is None or fuse is None:
+            post.add_into(hidden, y)
+            return
+        conv = part = None
+        after = ctx.extras.get("block_after")
+        if after is not None and isinstance(after[0], ParallelSublayersBlock) and after[0].mixer_input is not None:
+            part = after[0].mixer_input
+            conv = part.fusable(self.rt.ws.get("block.mixed", hidden.shape, self.rt.dtype), ctx, self._states(after[1])[1])
+        if not fuse(hidden, y, nxt, n, **({} if conv is None else {"conv": conv})):
+            post.add_into(hidden, y)
+            return
+        ctx.extras["stream.normed"] = (n.data_ptr(), id(nxt))
+        if conv is not None:
+            ctx.extras["stream.mixed"] = (conv[0].data_ptr(), id(part))

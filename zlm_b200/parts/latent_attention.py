@@ -13,7 +13,8 @@ With h the mixer's input, per token:
 Options: ``sink`` (a learned number per head, tensor ``sink`` [heads], whose exponential joins the softmax's denominator:
 it has no key and no value and is not scaled), ``gate`` (head h's output is multiplied by sigmoid(W_g h)_h, tensor ``g``
 [heads, hidden], one number per head from the mixer's own input) and ``chunk`` (a query sees only the keys of its own
-chunk of that many positions, counted from position 0).
+chunk of that many positions, counted from position 0) and ``q_rank`` (queries go through a latent of their own:
+q = W_uq (RMSNorm(W_dq h) * w_q), tensors ``dq`` [q_rank, hidden], ``dq.norm`` [q_rank], ``uq``; no ``q``).
 
 The cache record of a token is [c | kr] (``CacheRequest.token_shape``); a layer built with
 ``kv_proj=False`` has no W_dkv and reads the records of the schedule entry its own entry names
@@ -35,6 +36,7 @@ from typing import Any, Dict, Mapping, Optional
 
 import torch
 
+from ..kernels import pad_inner
 from ..registry import POSITION_ENCODINGS, lookup, register_mixer
 from .base import CacheRequest, LayerIO, Mixer, ParamSpec, StepContext
 
@@ -46,7 +48,7 @@ class LatentAttention(Mixer):
     def __init__(self, hidden_size: int, num_heads: int, head_dim: int, rot_dim: int, v_dim: int, kv_rank: int,
                  scale: float, norm_eps: float = 1e-6, window: int = 0,
                  position: Optional[Mapping[str, Any]] = None, kv_proj: bool = True, sink: bool = False,
-                 gate: bool = False, chunk: int = 0):
+                 gate: bool = False, chunk: int = 0, q_rank: int = 0):
         self.hidden = int(hidden_size)
         self.H, self.dn, self.dr, self.dv, self.r = int(num_heads), int(head_dim), int(rot_dim), int(v_dim), int(kv_rank)
         if min(self.H, self.dv, self.r) <= 0 or self.dn < 0 or self.dr < 0 or self.dn + self.dr <= 0:
@@ -54,6 +56,9 @@ class LatentAttention(Mixer):
         self.scale, self.eps, self.window = float(scale), float(norm_eps), int(window)
         self.kv_proj = bool(kv_proj)
         self.sink, self.gate, self.chunk = bool(sink), bool(gate), int(chunk)
+        self.qr = int(q_rank)                    # 0: queries straight from the input
+        if self.qr < 0:
+            raise ValueError(f"latent attention: q_rank={self.qr}")
         self.sinks: Optional[torch.Tensor] = None
         position = dict(position or {"kind": "none"})
         self.position = lookup(POSITION_ENCODINGS, "position encoding", position.pop("kind"))(**position)
@@ -68,10 +73,15 @@ class LatentAttention(Mixer):
 
     # ---- declarations -----------------------------------------------------
     def param_specs(self) -> Dict[str, ParamSpec]:
-        s = {"q": ParamSpec((self.Q, self.hidden)),
-             "uk": ParamSpec((self.H * self.dn, self.r)),
+        s = {"uk": ParamSpec((self.H * self.dn, self.r)),
              "uv": ParamSpec((self.H * self.dv, self.r)),
              "o": ParamSpec((self.hidden, self.H * self.dv))}
+        if self.qr:
+            s["dq"] = ParamSpec((self.qr, self.hidden))
+            s["dq.norm"] = ParamSpec((self.qr,), kind="vector", init="one_plus_normal")
+            s["uq"] = ParamSpec((self.Q, self.qr))
+        else:
+            s["q"] = ParamSpec((self.Q, self.hidden))
         if self.kv_proj:
             s["dkv"] = ParamSpec((self.R, self.hidden))
             s["dkv.norm"] = ParamSpec((self.r,), kind="vector", init="one_plus_normal")
@@ -94,14 +104,17 @@ class LatentAttention(Mixer):
         if not ctx.is_decode:
             return None
         from ..kernels import PAGE_TOKENS, attention_len_bucket
-        # (with chunks a query's keys span a chunk's pages at most, however long the sequence)
-        reach = min(ctx.max_len, self.chunk + PAGE_TOKENS) if self.chunk else ctx.max_len
+        # (behind a window, or in chunks, a query's keys span that many pages and one at most, however long the sequence)
+        spans = [n + PAGE_TOKENS for n in (self.chunk, self.window) if n]
+        reach = min([ctx.max_len] + spans)
         return ("latent_attention", attention_len_bucket(reach))
 
     def bind(self, params: Dict[str, torch.Tensor]) -> None:
         H, dn, dv, r = self.H, self.dn, self.dv, self.r
-        w_q = params.pop("q")
-        # one fused projection: rows [q | c_raw | kr_raw | gate], with rows of zeros up to a multiple of 8
+        # one fused projection: rows [q, or the query latent | c_raw | kr_raw | gate], with rows of zeros up to a multiple of 8
+        w_q = params.pop("dq" if self.qr else "q")
+        self.q_norm = params.pop("dq.norm") if self.qr else None
+        self.w_uq = pad_inner(params.pop("uq")) if self.qr else None
         rows = [w_q]
         if self.kv_proj:
             rows.append(params.pop("dkv"))
@@ -111,18 +124,20 @@ class LatentAttention(Mixer):
         self.g_off = sum(w.shape[0] for w in rows)
         if self.gate:
             rows.append(params.pop("g"))
-            n = self.g_off + H
-            if n % 8:
-                rows.append(torch.zeros((8 - n % 8, self.hidden), dtype=w_q.dtype, device=w_q.device))
+        n = sum(w.shape[0] for w in rows)
+        if (self.gate or self.qr) and n % 8:
+            rows.append(torch.zeros((8 - n % 8, self.hidden), dtype=w_q.dtype, device=w_q.device))
         self.w_in = torch.cat(rows, dim=0).contiguous() if len(rows) > 1 else w_q
         self.N_in = self.w_in.shape[0]
+        self.kv_off = self.qr or self.Q              # where the record's columns start in the fused projection
         if self.sink:
             self.sinks = params.pop("sink").float().contiguous()
         # per head: W_uk_h^T [r, dn] (folds into the query), W_uv_h [dv, r] (unfolds the output)
         self.w_uk_t = params.pop("uk").view(H, dn, r).transpose(1, 2).contiguous()
         self.w_uv = params.pop("uv").view(H, dv, r).contiguous()
         self.w_o = params.pop("o")
-        self.check_products(q=self.w_in, o=self.w_o)
+        self.w_o_even = pad_inner(self.w_o)          # the folded form's product: its input padded to a multiple of 8
+        self.check_products(q=self.w_in, o=self.w_o_even, uq=self.w_uq)
         # Whole prompts in bfloat16 may run unfolded (see ``_forward_unfolded``): the up-projections as one matrix
         # [W_uk | W_uv] applied to the step's latents, and W_o with a zero column for every column that pads a
         # head's values to the keys' width
@@ -138,11 +153,13 @@ class LatentAttention(Mixer):
             self.w_o_pad = pad.view(self.hidden, H * hd).contiguous()
 
     def tensors(self) -> Dict[str, torch.Tensor]:
-        out = {"q": self.w_in[: self.Q], "o": self.w_o,
+        out = {"dq" if self.qr else "q": self.w_in[: self.kv_off], "o": self.w_o,
                "uk": self.w_uk_t.transpose(1, 2).reshape(self.H * self.dn, self.r),
                "uv": self.w_uv.reshape(self.H * self.dv, self.r)}
+        if self.qr:
+            out["dq.norm"], out["uq"] = self.q_norm, self.w_uq[:, :self.qr]
         if self.kv_proj:
-            out["dkv"] = self.w_in[self.Q: self.Q + self.R]
+            out["dkv"] = self.w_in[self.kv_off: self.kv_off + self.R]
             out["dkv.norm"] = self.c_norm
         if self.sink:
             out["sink"] = self.sinks
@@ -168,13 +185,10 @@ class LatentAttention(Mixer):
             return
         qd = rt.ws.get("lat.qd", (T, self.N_in), rt.dtype)
         k.linear(qd, x, self.w_in)
-        q = qd[:, : self.Q]
-        q3 = qd.as_strided((T, H, self.Dq), (qd.stride(0), self.Dq, 1))
         # the folded query [q' | rotated part] of every head
         ql = rt.ws.get("lat.ql", (T, H, R), rt.dtype)
-        k.latent_prep(q, ql[:, :, r:], qd[:, self.Q: self.Q + R] if writes else None, self.c_norm, self.eps,
-                      self.position.inv_freq, self.position.n_rot, ctx.token_pos, ctx.token_slot,
-                      cache.block_table, cache.pool, H, dn, dr, r)
+        q = self._queries_and_records(qd, lambda q3: ql[:, :, r:], ctx, cache, writes)
+        q3 = q.as_strided((T, H, self.Dq), (q.stride(0), self.Dq, 1))
         if dn:
             k.head_linear(ql[:, :, :r], q3[:, :, :dn], self.w_uk_t)
         else:
@@ -184,11 +198,41 @@ class LatentAttention(Mixer):
         k.latent_attention(ol, ql.view(T, H * R), cache.pool, cache.block_table, ctx.token_pos, ctx.token_slot,
                            H, r, dr, self.scale, self.window, ctx, len_bucket=key[1] if key else None,
                            **self._options())
-        ov = rt.ws.get("lat.ov", (T, H * dv), rt.dtype)
-        k.head_linear(ov.view(T, H, dv), ol.view(T, H, r), self.w_uv)
+        ov = rt.ws.get("lat.ov", (T, self.w_o_even.shape[1]), rt.dtype)
+        if ov.shape[1] > H * dv:
+            ov[:, H * dv:].zero_()
+        heads = ov.as_strided((T, H, dv), (ov.stride(0), dv, 1))
+        k.head_linear(heads, ol.view(T, H, r), self.w_uv)
         if self.gate:
-            k.head_scalar_gate(ov.view(T, H, dv), qd[:, self.g_off: self.g_off + H])
-        k.linear(residual, ov, self.w_o, accumulate=True, defer=True)       # a norm reads the stream next
+            k.head_scalar_gate(heads, qd[:, self.g_off: self.g_off + H])
+        k.linear(residual, ov, self.w_o_even, accumulate=True, defer=True)  # a norm reads the stream next
+
+    def _queries_and_records(self, qd: torch.Tensor, rotated, ctx: StepContext, cache, writes: bool,
+                             rec_out: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """The heads' queries [T, H * (dim + rot_dim)] from the fused projection ``qd`` (through their latent, if they have
+        one), their rotated parts to where ``rotated(q3)`` says (q3: the queries by head), and the step's records to the
+        cache and to ``rec_out``."""
+        rt, k = self.rt, self.rt.k
+        T = qd.shape[0]
+        H, dn, dr, r, R = self.H, self.dn, self.dr, self.r, self.R
+        dkv = qd[:, self.kv_off: self.kv_off + R] if writes else None
+        freq, n_rot = self.position.inv_freq, self.position.n_rot
+        extra = {} if rec_out is None else {"rec_out": rec_out}
+        if self.qr:
+            cq = rt.ws.get("lat.cq", (T, self.w_uq.shape[1]), rt.dtype)
+            k.latent_down(cq, qd[:, :self.qr], self.q_norm, self.eps, dkv, self.c_norm, freq, n_rot, ctx.token_pos,
+                          ctx.token_slot, cache.block_table, cache.pool, dr, r, **extra)
+            q = rt.ws.get("lat.q", (T, (self.Q + 7) // 8 * 8), rt.dtype)[:, :self.Q]
+            k.linear(q, cq, self.w_uq)
+            dkv, extra = None, {}
+            if not dr:
+                return q
+        else:
+            q = qd[:, : self.Q]
+        q3 = q.as_strided((T, H, self.Dq), (q.stride(0), self.Dq, 1))
+        k.latent_prep(q, rotated(q3), dkv, self.c_norm, self.eps, freq, n_rot, ctx.token_pos, ctx.token_slot,
+                      cache.block_table, cache.pool, H, dn, dr, r, **extra)
+        return q
 
     def _options(self) -> Dict[str, Any]:
         """The attention kernels' words for the sink and the chunks (none of them for a mixer without)."""
@@ -229,19 +273,11 @@ class LatentAttention(Mixer):
         hd = dn + dr
         qd = rt.ws.get("lat.qd", (T, self.N_in), rt.dtype)
         k.linear(qd, x, self.w_in)
-        q = qd[:, : self.Q]
-        q3 = qd.as_strided((T, H, self.Dq), (qd.stride(0), self.Dq, 1))
         # rotated query parts in place; the records into their pages and, for this step's products, into plain rows
         # (a layer that reads another layer's records gathers them from the pages instead)
         rec = rt.ws.get("lat.rec", (T, R), rt.dtype)
-        if writes:
-            k.latent_prep(q, q3[:, :, dn:], qd[:, self.Q: self.Q + R], self.c_norm, self.eps,
-                          self.position.inv_freq, self.position.n_rot, ctx.token_pos, ctx.token_slot,
-                          cache.block_table, cache.pool, H, dn, dr, r, rec_out=rec)
-        else:
-            k.latent_prep(q, q3[:, :, dn:], None, self.c_norm, self.eps,
-                          self.position.inv_freq, self.position.n_rot, ctx.token_pos, ctx.token_slot,
-                          cache.block_table, cache.pool, H, dn, dr, r)
+        q = self._queries_and_records(qd, lambda q3: q3[:, :, dn:], ctx, cache, writes, rec_out=rec if writes else None)
+        if not writes:
             k.latent_gather(rec, cache.pool, cache.block_table, ctx.token_pos, ctx.token_slot)
         kv = rt.ws.get("lat.kv", (T, H * (dn + dv)), rt.dtype)
         k.linear(kv, rec[:, :r], self.w_ukv)

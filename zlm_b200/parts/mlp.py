@@ -10,6 +10,7 @@ from typing import Dict
 
 import torch
 
+from ..kernels import pad_inner
 from ..registry import register_feed_forward
 from .base import FeedForward, ParamSpec, StepContext
 
@@ -80,4 +81,39 @@ class SwiGLU(FeedForward):
                 k.gated_limit(act, gu, self.limit, self.alpha)
             else:
                 k.gated_act(act, gu, self.act)
+        k.linear(residual, act, self.w_down, accumulate=True, defer=True)      # a norm reads the stream next
+
+
+@register_feed_forward("poly_norm")
+class PolyNormMLP(FeedForward):
+    """W_down act(W_up x) without a gate: act(z) = a N(z) + b N(z^2) + c N(z^3) + e with powers taken element by element
+    and N dividing a token's vector of ff values by its root mean square (eps inside the root); (a, b, c, e) is the
+    checkpoint's vector ``act``."""
+
+    def __init__(self, hidden_size: int, intermediate_size: int, norm_eps: float):
+        self.hidden, self.inter, self.eps = int(hidden_size), int(intermediate_size), float(norm_eps)
+        if self.inter <= 0:
+            raise ValueError(f"poly_norm feed-forward: intermediate_size={self.inter}")
+
+    def param_specs(self) -> Dict[str, ParamSpec]:
+        return {"up_proj.weight": ParamSpec((self.inter, self.hidden)),
+                "down_proj.weight": ParamSpec((self.hidden, self.inter)),
+                "act": ParamSpec((4,), kind="vector", init="one_plus_normal")}
+
+    def bind(self, params: Dict[str, torch.Tensor]) -> None:
+        self.w_up = params.pop("up_proj.weight")
+        self.w_down = pad_inner(params.pop("down_proj.weight"))
+        self.coef = params.pop("act").contiguous()
+        self.check_products(up_proj=self.w_up, down_proj=self.w_down)
+
+    def tensors(self) -> Dict[str, torch.Tensor]:
+        return {"up_proj.weight": self.w_up, "down_proj.weight": self.w_down[:, :self.inter], "act": self.coef}
+
+    def forward(self, x: torch.Tensor, residual: torch.Tensor, ctx: StepContext) -> None:
+        rt, k = self.rt, self.rt.k
+        T, cols = x.shape[0], self.w_down.shape[1]
+        z = rt.ws.get("ffn.z", (T, cols), rt.dtype)[:, :self.inter]
+        k.linear(z, x, self.w_up)
+        act = rt.ws.get("ffn.act", (T, cols), rt.dtype)
+        k.poly_norm(act, z, self.coef, self.eps)
         k.linear(residual, act, self.w_down, accumulate=True, defer=True)      # a norm reads the stream next

@@ -9,7 +9,7 @@ from typing import Dict, List, Optional, Tuple
 import torch
 
 from ..config.spec import ConfigError, LayerSpec, ModelSpec, PartSpec
-from ..registry import (ARRANGEMENTS, EMBEDDINGS, FEED_FORWARDS, HEADS, MIXERS, NORMS, lookup)
+from ..registry import (ARRANGEMENTS, EMBEDDINGS, FEED_FORWARDS, HEADS, LAYER_INPUTS, MIXER_INPUTS, MIXERS, NORMS, lookup)
 from .base import (CacheRequest, LayerIO, ParamSpec, Part, Runtime, StateRequest, StepContext)
 
 
@@ -42,6 +42,10 @@ class DecoderModel:
             post = {name: (_build(NORMS, "norm", ps, size=H), ps)
                     for name, ps in (("mixer_post_norm", ls.mixer_post_norm), ("feed_forward_post_norm", ls.feed_forward_post_norm))
                     if ps is not None}
+            # (what the mixer's input passes through, what the layer reads beside the stream)
+            post.update({name: (_build(table, name.replace("_", " "), ps, hidden_size=H), ps)
+                         for name, table, ps in (("mixer_input", MIXER_INPUTS, ls.mixer_input),
+                                                 ("layer_input", LAYER_INPUTS, ls.layer_input)) if ps is not None})
             try:
                 block = lookup(ARRANGEMENTS, "block arrangement", ls.arrangement)(
                     hidden_size=H, mixer=mixer, feed_forward=ffn, mixer_norm=n1, feed_forward_norm=n2,
@@ -102,7 +106,9 @@ class DecoderModel:
         return [self.blocks[e.layer].mixer.cache_request() for e in self.spec.schedule]
 
     def state_requests(self) -> List[Optional[StateRequest]]:
-        return [self.blocks[e.layer].mixer.state_request() for e in self.spec.schedule]
+        """Per schedule entry: what the block asks for, or where it has no state beside its mixer's, the mixer."""
+        return [getattr(self.blocks[e.layer], "state_request", self.blocks[e.layer].mixer.state_request)()
+                for e in self.spec.schedule]
 
     def embedding_state_request(self) -> Optional[StateRequest]:
         """Per-sequence state that the embedding keeps (the token before a step's first one, for a table looked up by
@@ -140,8 +146,8 @@ class DecoderModel:
         hidden = rt.ws.get("model.hidden", (ctx.T, self.spec.hidden_size), torch.float32)
         # (the embedding writes the stream anew: whatever a run before this one, with the same context, noted about
         # copies of the stream, as the eager run before a capture does, no longer holds)
-        ctx.extras.pop("stream.rounded", None)
-        ctx.extras.pop("stream.normed", None)
+        for note in ("stream.rounded", "stream.normed", "stream.mixed"):
+            ctx.extras.pop(note, None)
         if getattr(self.embedding, "uses_step", False):
             self.embedding.forward(hidden, ctx.token_ids, ctx, embedding_io)
         else:
@@ -155,11 +161,12 @@ class DecoderModel:
             ctx.extras["norm_after_block"] = first() if first is not None else None
             first_part = getattr(nxt, "first_norm", None)
             ctx.extras["first_norm_after_block"] = first_part() if first_part is not None else None
+            ctx.extras["block_after"] = (nxt, ios[i + 1]) if nxt is not None else None
             self.blocks[e.layer].forward(hidden, ctx, io)
         ctx.extras["norm_after_block"] = None
-        ctx.extras["first_norm_after_block"] = None
-        ctx.extras.pop("stream.rounded", None)
-        ctx.extras.pop("stream.normed", None)
+        ctx.extras["first_norm_after_block"] = ctx.extras["block_after"] = None
+        for note in ("stream.rounded", "stream.normed", "stream.mixed"):
+            ctx.extras.pop(note, None)
         return hidden
 
     def logits(self, hidden: torch.Tensor, rows: torch.Tensor, n_rows: int,

@@ -1,4 +1,4 @@
-"""RMSNorm over rows of the fp32 residual stream.
+"""RMSNorm and LayerNorm over rows of the fp32 residual stream.
 
 y = (x * 1/sqrt(mean(x^2) + eps)) * w, weight used as it is
 (src/kernels/transformer/norm.zig:4-37).  ``scalar``: the checkpoint holds one gain for the whole
@@ -77,16 +77,38 @@ class RMSNorm(Norm):
         fused(stream, y, self.weight, self.eps, self.scale if self.layer_scale else None, cast_out=cast_out)
         return True
 
-
-    def add_into_then_norm(self, stream: torch.Tensor, y: torch.Tensor, nxt: Norm, out: torch.Tensor) -> bool:
-        """stream += norm(y) and out = nxt(stream) in one kernel, if both norms are of this kind without a scale of
-        their own and the kernel object has the kernel; the answer says whether it was done (else nothing was)."""
+    def add_into_then_norm(self, stream: torch.Tensor, y: torch.Tensor, nxt: Norm, out: torch.Tensor, conv=None) -> bool:
+        """stream += norm(y) and out = nxt(stream) in one kernel, if this norm has no scale of its own, ``nxt`` is such a
+        norm or a layer norm and the kernel object has the kernel; the answer says whether it was done (else nothing
+        was).  ``conv``: what the kernel object's ``norm_add_norm`` takes for a convolution of ``out`` in the same kernel."""
         fused = getattr(self.rt.k, "norm_add_norm", None)
-        if (fused is None or not isinstance(nxt, RMSNorm) or self.layer_scale or nxt.layer_scale or y.dtype != torch.float32
-                or self.size > getattr(self.rt.k, "NORM_ADD_NORM_MAX", 0)):
+        center = isinstance(nxt, LayerNorm)
+        if (fused is None or not (center or isinstance(nxt, RMSNorm)) or self.layer_scale or getattr(nxt, "layer_scale", False)
+                or y.dtype != torch.float32 or self.size > getattr(self.rt.k, "NORM_ADD_NORM_MAX", 0)):
             return False
-        fused(stream, y, self.weight, self.eps, out, nxt.weight, nxt.eps)
+        if not center and conv is None:
+            fused(stream, y, self.weight, self.eps, out, nxt.weight, nxt.eps)
+        else:
+            fused(stream, y, self.weight, self.eps, out, nxt.weight, nxt.eps, center=center, conv=conv)
         return True
+
+
+@register_norm("layer_norm")
+class LayerNorm(Norm):
+    """y = d / sqrt(mean(d^2) + eps) * w with d = x - mean(x): a weight per coordinate, no bias."""
+
+    def __init__(self, size: int, eps: float):
+        self.size, self.eps = int(size), float(eps)
+        self.weight: Optional[torch.Tensor] = None
+
+    def param_specs(self) -> Dict[str, ParamSpec]:
+        return {"weight": ParamSpec((self.size,), kind="vector", init="one_plus_normal")}
+
+    def bind(self, params: Dict[str, torch.Tensor]) -> None:
+        self.weight = params["weight"]
+
+    def forward(self, out: torch.Tensor, x: torch.Tensor, rows: Optional[torch.Tensor] = None) -> None:
+        self.rt.k.layernorm(out, x, self.weight, self.eps, rows)
 
 
 @register_norm("none")

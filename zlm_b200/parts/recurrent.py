@@ -1,4 +1,4 @@
-"""Two recurrent mixers whose whole memory of a sequence is a fixed-size fp32 state.
+"""Three recurrent mixers whose whole memory of a sequence is a fixed-size fp32 state.
 
 ``rglru``: a recurrent block with a real-gated linear recurrent unit.  Two branches of ``width`` channels read the
 mixer's input:
@@ -18,8 +18,15 @@ The state per sequence is S and the convolution's last ``conv_taps - 1`` inputs,
     S_t = diag(alpha_t) S_(t-1) + k_t v_t^T,   o_t = S_t^T q_t               per head
     out = W_o (rms_norm_per_head(o) * w_norm * silu(W_g x))                  w_norm [v_dim] shared by the heads
 
-The state per sequence is S [heads, head_dim, v_dim] fp32.  In both mixers everything between the projections and the
-output projection's input is fp32 whatever the compute dtype.
+The state per sequence is S [heads, head_dim, v_dim] fp32.
+
+``mingru``: a gated recurrence over ``width`` channels whose gates read the current token alone:
+
+    z = sigmoid(W_z x + b_z),  u = W_x x + b_x,  cand = u + 1/2 where u >= 0, sigmoid(u) where u < 0
+    S_t = (1 - z) S_(t-1) + z cand,  out = W_o (S * silu(W_g x))
+
+The state per sequence is S [width] fp32.  In all of them everything between the projections and the output
+projection's input is fp32 whatever the compute dtype.
 """
 from __future__ import annotations
 
@@ -27,6 +34,7 @@ from typing import Dict, Optional
 
 import torch
 
+from ..kernels import pad_inner
 from ..registry import register_mixer
 from .base import LayerIO, Mixer, ParamSpec, StateRequest, StepContext
 
@@ -145,3 +153,47 @@ class GatedLinearAttention(Mixer):
         y = rt.ws.get("gla.gated", (T, VV), rt.dtype)
         k.norm_gate(y, o, proj[:, 2 * QK + VV: 2 * QK + 2 * VV], self.H, self.V, "head", self.w_norm, self.eps, self.gate)
         k.linear(residual, y, self.w_o, accumulate=True, defer=True)       # a norm reads the stream next
+
+
+@register_mixer("mingru")
+class MinGRU(Mixer):
+    reads_input_by_products = True       # x goes into the fused projection and nowhere else
+
+    def __init__(self, hidden_size: int, width: int):
+        self.hidden, self.W = int(hidden_size), int(width)
+        if self.W <= 0:
+            raise ValueError(f"mingru: {self.W} channels")
+
+    def param_specs(self) -> Dict[str, ParamSpec]:
+        W, K = self.W, self.hidden
+        return {"z_proj.weight": ParamSpec((W, K)), "z_proj.bias": ParamSpec((W,), kind="vector", init="zeros"),
+                "x_proj.weight": ParamSpec((W, K)), "x_proj.bias": ParamSpec((W,), kind="vector", init="zeros"),
+                "g_proj.weight": ParamSpec((W, K)), "o_proj.weight": ParamSpec((K, W))}
+
+    def state_request(self) -> Optional[StateRequest]:
+        return StateRequest((self.W,), torch.float32)
+
+    def bind(self, params: Dict[str, torch.Tensor]) -> None:
+        # one fused projection: rows [z | x | g]
+        self.w_in = torch.cat([params.pop(f"{n}_proj.weight") for n in ("z", "x", "g")], dim=0).contiguous()
+        self.b_z, self.b_x = params.pop("z_proj.bias"), params.pop("x_proj.bias")
+        if self.b_z.dtype != self.b_x.dtype:
+            self.b_z, self.b_x = self.b_z.float(), self.b_x.float()
+        self.w_o = pad_inner(params.pop("o_proj.weight"))
+        self.check_products(in_proj=self.w_in, o_proj=self.w_o)
+
+    def tensors(self) -> Dict[str, torch.Tensor]:
+        W = self.W
+        return {"z_proj.weight": self.w_in[:W], "x_proj.weight": self.w_in[W:2 * W], "g_proj.weight": self.w_in[2 * W:],
+                "z_proj.bias": self.b_z, "x_proj.bias": self.b_x, "o_proj.weight": self.w_o[:, :W]}
+
+    def forward(self, x: torch.Tensor, residual: torch.Tensor, ctx: StepContext, io: LayerIO) -> None:
+        rt, k, W = self.rt, self.rt.k, self.W
+        T, cols = x.shape[0], self.w_o.shape[1]
+        proj = rt.ws.get("mingru.proj", (T, 3 * W), rt.dtype)
+        k.linear(proj, x, self.w_in)
+        gated = rt.ws.get("mingru.gated", (T, cols), rt.dtype)
+        if cols > W:
+            gated[:, W:].zero_()
+        k.mingru(gated[:, :W], proj, 0, W, 2 * W, self.b_z, self.b_x, io.state, ctx)
+        k.linear(residual, gated, self.w_o, accumulate=True, defer=True)       # a norm reads the stream next

@@ -27,6 +27,8 @@ POSITION_ENCODINGS: Dict[str, Any] = {}
 ARRANGEMENTS: Dict[str, Any] = {}
 EMBEDDINGS: Dict[str, Any] = {}
 HEADS: Dict[str, Any] = {}
+MIXER_INPUTS: Dict[str, Any] = {}
+LAYER_INPUTS: Dict[str, Any] = {}
 
 
 def _register(table: Dict[str, Any], what: str, name: str):
@@ -68,6 +70,14 @@ def register_embedding(kind: str):
 
 def register_head(kind: str):
     return _register(HEADS, "head", kind)
+
+
+def register_mixer_input(kind: str):
+    return _register(MIXER_INPUTS, "mixer input", kind)
+
+
+def register_layer_input(kind: str):
+    return _register(LAYER_INPUTS, "layer input", kind)
 
 
 def lookup(table: Dict[str, Any], what: str, kind: str):
