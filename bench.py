@@ -606,13 +606,62 @@ SUDUPEL_SIZES = {
     "small": (_sudupel(1024, 8, 2, 512, 3072, 16, 2, 1536, "wplwpp", 32768), _twin(1024, 8, 2, 3072, 6, 32768)),
     "wide": (_sudupel(4096, 32, 8, 4096, 12288, 16, 2, 6144, "wplp", 32768), _twin(4096, 32, 8, 12288, 4, 32768)),
 }
+def _murilix(width, heads, dim, rot, vdim, q_rank, rank, window, gru, ff, experts, top, expert_ff, taps, side, kinds, vocab):
+    """Layers of kind "g" (the gated recurrence), "L" (latent attention with latents of its own) and "l" (latent attention
+    over the latents of the last "L" layer before it); the first layer's feed-forward dense, the others routed."""
+    mixer = {"heads": heads, "dim": dim, "rot_dim": rot, "vdim": vdim, "q_rank": q_rank, "kv_rank": rank,
+             "scale": (dim + rot) ** -0.5, "mask": {"size": window}, "rot": {"base": 10000.0, "dims": rot}}
+    moe = {"kind": "moe", "expert": {"ff": expert_ff}, "router": {"experts": experts, "top": top}}
+    layers, last = [], None
+    for i, k in enumerate(kinds):
+        m = {"width": gru} if k == "g" else dict(mixer)
+        if k == "L":
+            last = i
+        elif k == "l":
+            m["kv_from"] = last
+        layers.append({"type": "mingru" if k == "g" else "latent_attention", "mixer": m,
+                       "mlp": {"kind": "dense", "ff": ff} if i == 0 else moe})
+    return {"architecture": "Murilix", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "embedding": {"scale": width ** 0.5},
+            "canon": {"taps": taps}, "token_side": {"dim": side}, "layers": layers}
+
+
+def _nuvilorn_twin(width, heads, dim, rot, vdim, rank, ff, experts, top, expert_ff, kinds, vocab):
+    """A Nuvilorn model of the same width, heads, latents, layers (every one latent attention; those that read another
+    layer's latents, the same), experts and vocabulary; its ungated experts and gated dense layer do as many multiply-adds."""
+    mixer = {"heads": heads, "dim": dim, "rot_dim": rot, "vdim": vdim, "kv_rank": rank,
+             "scale": (dim + rot) ** -0.5, "rot": {"base": 10000.0, "dims": rot}}
+    moe = {"kind": "moe", "expert": {"ff": expert_ff * 3 // 2}, "router": {"experts": experts, "top": top}}
+    layers, last = [], None
+    for i, k in enumerate(kinds):
+        m = dict(mixer)
+        if k == "l":
+            m["kv_from"] = last
+        else:
+            last = i
+        layers.append({"type": "latent_attention", "mixer": m, "mlp": {"kind": "dense", "ff": ff * 2 // 3} if i == 0 else moe})
+    return {"architecture": "Nuvilorn", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "layers": layers}
+
+
+# Murilix: the three kinds of layer, windows that cover the run (so that attention does the work of the twin's) or a quarter
+# of it ("small")
+MURILIX_SIZES = {
+    # 16 heads of 128 + 64 over latents of 512, queries through 768, recurrences of the model's width, 64 experts of 1024
+    # (6 a token), 256 side columns a layer
+    "lite": (_murilix(2048, 16, 128, 64, 128, 768, 512, 4096, 2048, 9216, 64, 6, 1024, 4, 256, "gLlgLl", 32768),
+             _nuvilorn_twin(2048, 16, 128, 64, 128, 512, 9216, 64, 6, 1024, "LLlLLl", 32768)),
+    "small": (_murilix(1024, 8, 64, 32, 64, 384, 256, 512, 1536, 4608, 32, 4, 512, 3, 128, "gLlgLl", 32768),
+              _nuvilorn_twin(1024, 8, 64, 32, 64, 256, 4608, 32, 4, 512, "LLlLLl", 32768)),
+    "wide": (_murilix(4096, 32, 128, 64, 128, 1536, 512, 4096, 4096, 18432, 32, 2, 2048, 4, 256, "gLlg", 32768),
+             _nuvilorn_twin(4096, 32, 128, 64, 128, 512, 18432, 32, 2, 2048, "LLlL", 32768)),
+}
 DESIGNS = {"nuvilorn": ("Nuvilorn", DESIGN_SIZES), "zekazen": ("Zekazen", ZEKAZEN_SIZES),
-           "lodevik": ("Lodevik", LODEVIK_SIZES), "sudupel": ("Sudupel", SUDUPEL_SIZES)}
+           "lodevik": ("Lodevik", LODEVIK_SIZES), "sudupel": ("Sudupel", SUDUPEL_SIZES),
+           "murilix": ("Murilix", MURILIX_SIZES)}
 
 
 def design_comparison(args) -> int:
     """Prefill of 2,048 tokens and decode at batch ``--batch`` from 2,048-token prompts, device-timed, for
-    the design named by ``--design`` and for its Qwen3-dense twin at each of the design's sizes, with every
+    the design named by ``--design`` and for its twin (Qwen3 dense, or the design it is closest to) at each of the design's sizes, with every
     operation of both steps (CUDA events; decode operations as graphs of one step's calls); one JSON line."""
     import torch
     from zlm_b200 import Engine, StepEntry
@@ -624,11 +673,13 @@ def design_comparison(args) -> int:
     B, L, steps, warmup = args.batch, PROMPT_LEN, min(args.steps, 64), max(3, args.warmup)
     g = torch.Generator().manual_seed(0)
     design, sizes = DESIGNS[args.design]
-    out = {"metric": f"prefill and decode tokens/s of {design} beside Qwen3 dense at equal sizes", "unit": "tokens/s",
+    twin = "qwen3_twin" if "architectures" in next(iter(sizes.values()))[1] else "nuvilorn_twin"
+    beside = {"qwen3_twin": "Qwen3 dense", "nuvilorn_twin": "Nuvilorn"}[twin]
+    out = {"metric": f"prefill and decode tokens/s of {design} beside {beside} at equal sizes", "unit": "tokens/s",
            "dtype": "bf16", "data": "synthetic", "batch": B, "prompt_len": L, "peaks": pk, "sizes": {}}
     for name in ([args.design_size] if args.design_size else list(sizes)):
         rec = {}
-        for which, d in zip((args.design, "qwen3_twin"), sizes[name]):
+        for which, d in zip((args.design, twin), sizes[name]):
             cfg = config_from_dict(d)
             eng = Engine.from_random(cfg, seed=0, dtype="bfloat16", device="cuda:0", max_tokens=B * (L + 256),
                                      max_batch=B, max_seq_len=L + 256, max_step_tokens=B * L)
@@ -714,7 +765,8 @@ def main() -> int:
     ap.add_argument("--no-other-sizes", action="store_true",
                     help="leave out the Qwen3-0.6B and Qwen3-32B sizes that the default run adds under points")
     ap.add_argument("--design", choices=sorted(DESIGNS),
-                    help="instead of the headline run: that design beside its Qwen3-dense twin at a few layer sizes")
+                    help="instead of the headline run: that design beside its twin (Qwen3 dense, or the design it is "
+                         "closest to) at a few layer sizes")
     ap.add_argument("--design-size", choices=sorted(DESIGN_SIZES), default=None, help="with --design: one of the sizes only")
     args = ap.parse_args()
     if args.impl == "reference":

@@ -171,7 +171,7 @@ def forward(config: Mapping, tensors: Mapping[str, torch.Tensor], tokens: List[i
     dim = int(config["token_side"]["dim"])
     T = len(tokens)
     ids, positions = torch.tensor(tokens), torch.arange(T)
-    x = _w(tensors, "embed")[ids] * float(config["embedding"]["scale"])
+    x = _w(tensors, "embed")[ids] * float((config.get("embedding") or {}).get("scale", 1.0))
     side = _w(tensors, "side.embed")[ids]
     streams, records = [], {}
     closest = torch.full((T,), math.inf, dtype=F64)

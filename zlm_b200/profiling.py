@@ -286,9 +286,41 @@ class ProfilingKernels:
         return self._timed(kind, n, 6.0 * T * heads * dim * v_dim, self.k.linear_attention, o, proj, q_off, k_off, v_off,
                            alpha, head_decay, state, plan, heads, dim, v_dim, *args, **kw)
 
-    def norm_add_norm(self, stream, y, w1, eps1, out2, w2, eps2):
-        return self._timed("sublayer norm+add+next norm", 3 * _nbytes(stream) + _nbytes(out2), 0, self.k.norm_add_norm,
-                           stream, y, w1, eps1, out2, w2, eps2)
+    def norm_add_norm(self, stream, y, w1, eps1, out2, w2, eps2, center=False, conv=None):
+        n, name = 3 * _nbytes(stream) + _nbytes(out2), "sublayer norm+add+next norm"
+        if conv is not None:
+            n, name = n + (2 * conv[1].shape[0] - 1) * _nbytes(out2) + _nbytes(conv[1]), name + "+conv"
+        kw = {} if not center and conv is None else {"center": center, "conv": conv}
+        return self._timed(name, n, 0, self.k.norm_add_norm, stream, y, w1, eps1, out2, w2, eps2, **kw)
+
+    # a layer norm, the mixer's input convolved, a polynomial of normed powers, a gated recurrence, the tokens' side rows
+    def layernorm(self, out, x, w, eps, rows=None):
+        R, H = out.shape
+        return self._timed("layernorm", R * H * 4 + _nbytes(out) + _nbytes(w), 0, self.k.layernorm, out, x, w, eps, rows)
+
+    def input_conv(self, out, h, w, state, plan):
+        n = 2 * _nbytes(h) + _nbytes(w) + 2 * plan.R * (w.shape[0] - 1) * h.shape[1] * h.element_size()
+        return self._timed("mixer input convolved", n, 0, self.k.input_conv, out, h, w, state, plan)
+
+    def poly_norm(self, out, z, coef, eps):
+        return self._timed("polynomial of normed powers", _nbytes(out) + z.numel() * z.element_size(), 0, self.k.poly_norm,
+                           out, z, coef, eps)
+
+    def mingru(self, out, proj, *args, **kw):
+        T, W = out.shape
+        return self._timed("gated recurrence (mingru)", 4 * T * W * out.element_size(), 0, self.k.mingru, out, proj, *args, **kw)
+
+    def token_gate(self, g, z, *args):
+        return self._timed("tokens' side rows gated", 3 * _nbytes(g), 0, self.k.token_gate, g, z, *args)
+
+    def token_gate_few(self, g, x, w, *args):
+        return self._timed("side gate product+gelu+rows", _nbytes(w) + _nbytes(x) + 2 * _nbytes(g), 2.0 * x.shape[0] * w.numel(),
+                           self.k.token_gate_few, g, x, w, *args)
+
+    def latent_down(self, cq, down, q_weight, eps, dkv=None, *args, **kw):
+        n = 2 * _nbytes(cq) + 2 * _nbytes(dkv)
+        return self._timed("query latent norm" + ("+latent norm+rope+cache_write" if dkv is not None else ""), n, 0,
+                           self.k.latent_down, cq, down, q_weight, eps, dkv, *args, **kw)
 
     def scaled_sum(self, out, a, alpha, b, beta, accumulate=True):
         return self._timed("two sides summed", 3 * _nbytes(out), 0, self.k.scaled_sum, out, a, alpha, b, beta, accumulate)
@@ -304,7 +336,8 @@ class ProfilingKernels:
 
     # latent attention and routed experts
     def latent_prep(self, q, q_rot, dkv, *args, **kw):
-        n = _nbytes(q) + _nbytes(q_rot) + 2 * _nbytes(dkv)
+        # (only the rotated parts of q are read)
+        n = 2 * _nbytes(q_rot) + 2 * _nbytes(dkv)
         return self._timed("latent norm+rope+cache_write", n, 0, self.k.latent_prep, q, q_rot, dkv, *args, **kw)
 
     def latent_gather(self, rec, *args):
