@@ -203,3 +203,32 @@ def test_a_batch_of_many_requests_through_captured_steps(tmp_path, name):
     alone = [eng.generate([p], max_tokens=10).tokens[0] for p in ps]
     assert together == alone
     eng.check(sync=True)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("name", NAMES)
+def test_sublayers_side_by_side_give_the_bits_they_give_in_turn(tmp_path, name, dtype, monkeypatch):
+    """Decode steps of 3 and of 20 rows (the many-token products leave shares of sums in scratch memory that the two
+    sides must not share), captured and not: the logits are the same bits with the two sublayers on two streams."""
+    from zlm_b200 import StepEntry
+    from zlm_b200.parts.block import ParallelSublayersBlock
+    from zlm_b200.sampling import SamplingParams
+    eng, cfg, _ = build(tmp_path, name, dtype, max_tokens=64 * 64, max_batch=32)
+    for rows in (3, 20):
+        ps = prompts(cfg["vocab"], [5 + 3 * i for i in range(rows)], seed=rows)
+        got = {}
+        for mode in (True, False):
+            monkeypatch.setattr(ParallelSublayersBlock, "side_by_side", mode)
+            eng.decoder.graphs.clear()
+            slots = [eng.new_sequence() for _ in ps]
+            eng.step([StepEntry(s, p, []) for s, p in zip(slots, ps)])
+            out = [eng.step([StepEntry(s, [7], [0]) for s in slots]).clone()]
+            toks = [3] * rows
+            for _ in range(4):
+                toks = eng.decoder.step(slots, toks, SamplingParams()).tolist()
+                out.append(eng.decoder.last_logits.clone())
+            got[mode] = torch.stack(out)
+            for s in slots:
+                eng.release(s)
+        assert torch.equal(got[True], got[False]), f"{name}: {rows} rows"
+    eng.check(sync=True)

@@ -178,7 +178,7 @@ def test_query_latents_and_records_from_one_kernel(dtype):
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("width", [27, 48, 300])
 def test_gated_recurrence_remembers_from_far_back(tmp_path, dtype, width):
-    """Gates near 0.01: 500 tokens whole (in pieces side by side), in portions, then token by token; two sequences side
+    """Gates near 0.01: 500 tokens whole (a cluster's warps side by side), in portions, then token by token; two sequences side
     by side; a slot used again starts from zero."""
     from zlm_b200 import StepEntry
     cfg = one_layer({"width": width}, dense(32))
@@ -194,16 +194,16 @@ def test_gated_recurrence_remembers_from_far_back(tmp_path, dtype, width):
     assert_rows_close(run_cut(eng, a, [500]), want, dtype, "whole")
     assert_rows_close(run_cut(eng, a, [1, 2, 1, 3, 250, 2, 200], then_single=41), want, dtype, "portions, then single tokens")
     s1, s2 = eng.new_sequence(), eng.new_sequence()
-    got = eng.step([StepEntry(s1, b, [36]), StepEntry(s2, a[:200], [99, 199])]).clone()          # (pieces, unequal sequences)
+    got = eng.step([StepEntry(s1, b, [36]), StepEntry(s2, a[:200], [99, 199])]).clone()          # (clusters, unequal sequences)
     assert_rows_close(got, torch.stack([P.forward(cfg, ref, b)[0][36], want[99], want[199]]), dtype, "side by side")
     got = eng.step([StepEntry(s1, a[:5], []), StepEntry(s2, a[200:210], [9])]).clone()
-    assert_rows_close(got, want[209:210], dtype, "going on from the pieces' state")
+    assert_rows_close(got, want[209:210], dtype, "going on from the cluster's state")
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("pieces", [False, True])
-@pytest.mark.parametrize("W,lens", [(5, [1, 1]), (64, [200, 1, 33]), (130, [31, 32, 65, 700]), (128, [1100])])
-def test_gated_recurrence_kernel(dtype, pieces, W, lens):
+@pytest.mark.parametrize("cluster", [False, True])
+@pytest.mark.parametrize("W,lens", [(5, [1, 1]), (64, [200, 1, 33]), (130, [31, 32, 65, 700]), (128, [1100]), (66, [2100, 7, 1024])])
+def test_gated_recurrence_kernel(dtype, cluster, W, lens):
     """The kernel alone from states that are not zero: candidates on both sides of u = 0 (and at it), gates saturated
     either way, columns in any order inside wider rows, slots not in order."""
     from zlm_b200.kernels import get_kernels
@@ -222,7 +222,7 @@ def test_gated_recurrence_kernel(dtype, pieces, W, lens):
     state = torch.randn(R, W, generator=g)
     st = state.cuda().clone()
     out = torch.empty(T, W + 2, dtype=dt, device="cuda")[:, :W]
-    k.mingru(out, proj.cuda(), off["z"], off["x"], off["g"], bz.cuda(), bx.cuda(), st, plan_for(lens, [3] * R, slots), pieces=pieces)
+    k.mingru(out, proj.cuda(), off["z"], off["x"], off["g"], bz.cuda(), bx.cuda(), st, plan_for(lens, [3] * R, slots), cluster=cluster)
     p, at = proj.to(F64), 0
     tol = 2e-5 if dtype == "float32" else 8e-3
     for r, n in enumerate(lens):
@@ -272,6 +272,27 @@ def test_input_convolution_kernel(dtype, taps, C):
     assert at == total or at == [60, 9, 31]
     for r in range(3):
         assert_rows_close(torch.cat(got[r]), want[r], dtype, f"sequence {r}", 1e-5 if dtype == "float32" else 6e-3)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("taps", [2, 3, 4, 6])
+def test_input_convolution_of_many_tokens(dtype, taps):
+    """700 tokens of five sequences (runs of tokens that cross from one into the next, sequences shorter than the
+    convolution among them), from states that are not zero."""
+    from zlm_b200.kernels import get_kernels
+    dt = torch.float32 if dtype == "float32" else torch.bfloat16
+    g = torch.Generator().manual_seed(taps)
+    C, lens, slots = 136, [301, 1, 2, 390, 6], [3, 0, 4, 1, 2]
+    w = (torch.randn(C, taps, generator=g) * 0.8).to(dt)
+    st0 = torch.randn(5, taps - 1, C, generator=g).to(dt)
+    h, st = torch.randn(sum(lens), C, generator=g).to(dt), st0.cuda()
+    out = torch.empty(sum(lens), C, dtype=dt, device="cuda")
+    get_kernels().input_conv(out, h.cuda(), w.t().contiguous().cuda(), st, plan_for(lens, [9] * 5, slots))
+    for r, (x, o) in enumerate(zip(h.split(lens), out.cpu().split(lens))):
+        ext = torch.cat([st0[slots[r]], x])
+        want = x.to(F64) + P.causal_conv(ext.to(F64), w.to(F64))[taps - 1:]
+        assert_rows_close(o, want, dtype, f"sequence {r}", 1e-5 if dtype == "float32" else 6e-3)
+        assert torch.equal(st[slots[r]].cpu(), ext[len(ext) - (taps - 1):])
 
 
 @pytest.mark.parametrize("dtype", DTYPES)

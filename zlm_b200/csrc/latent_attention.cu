@@ -135,7 +135,9 @@ extern "C" int zlm_latent_prep(const void* q, int q_stride, void* qo, int qo_str
 }
 
 // Queries through a latent of their own: cq[t, :qr] = RMSNorm(down[t, :qr]) * qw (columns of cq from qr up to cq_cols
-// become zeros), and, where the projection has them (dkv not null), the token's record as above.  One block per token.
+// become zeros), and, where the projection has them (dkv not null), the token's record as above.  A block per token and
+// task: the query latents' in the grid's first row, the records' in the second.
+#define LD_KEEP 8            // a latent's first 1,024 columns stay in registers between the sum and the scaling
 template <typename TA>
 __global__ void __launch_bounds__(128)
 latent_down_kernel(TA* __restrict__ cq, int cq_stride, int cq_cols, const TA* __restrict__ down, int down_stride, int qr, VecW qw,
@@ -146,34 +148,45 @@ latent_down_kernel(TA* __restrict__ cq, int cq_stride, int cq_cols, const TA* __
     __shared__ float cs[2][256];
     pdl_trigger();
     const int t = blockIdx.x;
-    int pos = 0, slot = 0;
-    if (dkv) {
+    if (blockIdx.y == 1) {
         if (!ZLM_CHK(token_pos + t, 4) || !ZLM_CHK(token_slot + t, 4)) return;
-        pos = token_pos[t];
-        slot = token_slot[t];
+        const int pos = token_pos[t], slot = token_slot[t];
         for (int i = threadIdx.x; i < n_rot / 2; i += blockDim.x) {
             float s, c;
             sincosf((float)pos * inv_freq[i], &s, &c);
             cs[0][i] = c;
             cs[1][i] = s;
         }
+        pdl_wait();
+        __syncthreads();
+        write_record(dkv + (size_t)t * down_stride, cw, eps, cs[0], cs[1], n_rot, pos, slot, block_table, table_stride, pool, dr, r,
+                     rec_out ? rec_out + (size_t)t * rec_stride : nullptr, red);
+        return;
     }
     pdl_wait();
-    __syncthreads();
     const TA* src = down + (size_t)t * down_stride;
     TA* o = cq + (size_t)t * cq_stride;
     if (!ZLM_CHK(src, (size_t)qr * sizeof(TA)) || !ZLM_CHK(o, (size_t)cq_cols * sizeof(TA))) return;
+    float keep[LD_KEEP];
     float ss = 0.f;
-    for (int i = threadIdx.x; i < qr; i += blockDim.x) {
+#pragma unroll
+    for (int j = 0; j < LD_KEEP; ++j) {
+        const int i = threadIdx.x + j * 128;
+        keep[j] = i < qr ? to_f32(src[i]) : 0.f;
+        ss = fmaf(keep[j], keep[j], ss);
+    }
+    for (int i = threadIdx.x + LD_KEEP * 128; i < qr; i += 128) {
         const float a = to_f32(src[i]);
         ss = fmaf(a, a, ss);
     }
     ss = block_sum(ss, red);
     const float inv = 1.0f / sqrtf(ss / (float)qr + eps);
-    for (int i = threadIdx.x; i < cq_cols; i += blockDim.x) o[i] = from_f32<TA>(i < qr ? (to_f32(src[i]) * inv) * qw[i] : 0.f);
-    if (dkv)
-        write_record(dkv + (size_t)t * down_stride, cw, eps, cs[0], cs[1], n_rot, pos, slot, block_table, table_stride, pool, dr, r,
-                     rec_out ? rec_out + (size_t)t * rec_stride : nullptr, red);
+#pragma unroll
+    for (int j = 0; j < LD_KEEP; ++j) {
+        const int i = threadIdx.x + j * 128;
+        if (i < cq_cols) o[i] = from_f32<TA>(i < qr ? (keep[j] * inv) * qw[i] : 0.f);
+    }
+    for (int i = threadIdx.x + LD_KEEP * 128; i < cq_cols; i += 128) o[i] = from_f32<TA>(i < qr ? (to_f32(src[i]) * inv) * qw[i] : 0.f);
 }
 
 extern "C" int zlm_latent_down(void* cq, int cq_stride, int cq_cols, const void* down, int down_stride, int dtype, int qr,
@@ -192,7 +205,7 @@ extern "C" int zlm_latent_down(void* cq, int cq_stride, int cq_cols, const void*
     }
     const VecW q{qw, qw_dtype}, w{cw ? cw : qw, cw ? cw_dtype : qw_dtype};
 #define ZLM_LD(TA)                                                                                                        \
-    zlm_launch(latent_down_kernel<TA>, T, 128, 0, st, (TA*)cq, cq_stride, cq_cols, (const TA*)down, down_stride, qr, q,       \
+    zlm_launch(latent_down_kernel<TA>, dim3(T, dkv ? 2 : 1), 128, 0, st, (TA*)cq, cq_stride, cq_cols, (const TA*)down, down_stride, qr, q,       \
                (const TA*)dkv, w, eps, inv_freq, n_rot, token_pos, token_slot, block_table, table_stride, (TA*)pool, dr, r,  \
                (TA*)rec_out, rec_stride)
     if (dtype == ZLM_DTYPE_F32) ZLM_LD(float);

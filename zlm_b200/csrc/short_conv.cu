@@ -537,26 +537,14 @@ extern "C" int zlm_norm_gate(void* out, int out_stride, const float* o, const vo
 // ---------------------------------------------------------------------------- a mixer's input convolved
 // out[t] = h[t] + sum_j w[j] * h_(t - taps + 1 + j), per channel, zeros before the sequence's start; w [taps][C].  The
 // rows of earlier steps come from the state, [slots][taps-1][C] in the element type, oldest first (zeros in a new slot).
-// The threads of a sequence's first token of the step do its first taps - 1 tokens, the only ones that read the state,
-// and then bring the state up to date: nobody else touches it.
+// Whoever does a sequence's first token of the step does its first taps - 1 tokens, the only ones that read the state,
+// and then brings the state up to date: nobody else touches it.
+
+// a sequence's first tokens of the step, [0, last), and its state after the step's n; VEC channels from c on
 template <typename TA, int VEC>
-__global__ void __launch_bounds__(128)
-input_conv_kernel(TA* __restrict__ out, const TA* __restrict__ h, const TA* __restrict__ w, TA* state,
-                  const int* __restrict__ token_seq, const int* __restrict__ cu_seqlens, const int* __restrict__ seq_slot,
-                  int C, int taps) {
-    pdl_trigger();
-    const int t = blockIdx.x, c = (blockIdx.y * blockDim.x + threadIdx.x) * VEC;
-    pdl_wait();
-    if (c >= C || !ZLM_CHK(token_seq + t, 4)) return;
-    const int r = token_seq[t];
-    if (!ZLM_CHK(cu_seqlens + r, 8) || !ZLM_CHK(seq_slot + r, 4)) return;
-    const int row0 = cu_seqlens[r], n = cu_seqlens[r + 1] - row0, i = t - row0;
-    if (i > 0 && i < taps - 1) return;
-    const int last = i == 0 ? max(1, min(n, taps - 1)) : i + 1;
-    TA* st = taps > 1 ? state + (size_t)seq_slot[r] * (taps - 1) * C + c : nullptr;
-    if (i == 0 && st && !ZLM_CHK(st, ((size_t)(taps - 2) * C + VEC) * sizeof(TA))) return;
-    if (!ZLM_CHK(w + c, ((size_t)(taps - 1) * C + VEC) * sizeof(TA))) return;
-    for (int s = i; s < last; ++s) {
+__device__ __forceinline__ void input_conv_head(TA* __restrict__ out, const TA* __restrict__ h, const TA* __restrict__ w, TA* st,
+                                                int row0, int n, int last, int C, int c, int taps) {
+    for (int s = 0; s < last; ++s) {
         float a[VEC], u[VEC], k[VEC];
 #pragma unroll
         for (int v = 0; v < VEC; ++v) a[v] = u[v] = 0.f;
@@ -574,7 +562,6 @@ input_conv_kernel(TA* __restrict__ out, const TA* __restrict__ h, const TA* __re
         TA* o = out + (size_t)(row0 + s) * C + c;
         if (ZLM_CHK(o, VEC * sizeof(TA))) store_vec<TA, VEC>(o, a);
     }
-    if (i > 0 || taps == 1) return;
     // the newest taps - 1 rows, in ascending order: a row taken from the old state lies further on than the one written
     for (int m = 0; m < taps - 1; ++m) {
         const int p = n - (taps - 1) + m;
@@ -586,18 +573,100 @@ input_conv_kernel(TA* __restrict__ out, const TA* __restrict__ h, const TA* __re
     }
 }
 
+// A block: a run of RUN tokens and 128 x VEC channels.  With TAPS > 0 the rows the run needs are loaded at once and stay
+// in registers; TAPS 0: any number of taps, row by row.
+template <typename TA, int VEC, int TAPS, int RUN>
+__global__ void __launch_bounds__(128)
+input_conv_kernel(TA* __restrict__ out, const TA* __restrict__ h, const TA* __restrict__ w, TA* state,
+                  const int* __restrict__ token_seq, const int* __restrict__ cu_seqlens, const int* __restrict__ seq_slot,
+                  int T, int C, int any_taps) {
+    const int taps = TAPS > 0 ? TAPS : any_taps;
+    pdl_trigger();
+    const int t0 = blockIdx.x * RUN, c = (blockIdx.y * blockDim.x + threadIdx.x) * VEC;
+    if (c >= C || !ZLM_CHK(w + c, ((size_t)(taps - 1) * C + VEC) * sizeof(TA))) return;
+    float k[TAPS > 0 ? TAPS : 1][VEC], u[TAPS > 0 ? RUN + TAPS - 1 : 1][VEC];
+    if (TAPS > 0)
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) load_vec<TA, VEC>(w + (size_t)j * C + c, k[j]);
+    pdl_wait();
+    if (TAPS > 0)
+#pragma unroll
+        for (int i = 0; i < RUN + TAPS - 1; ++i) {
+            const int t = t0 - (TAPS - 1) + i;
+            if (t >= 0 && t < T && ZLM_CHK(h + (size_t)t * C + c, VEC * sizeof(TA))) {
+                load_vec<TA, VEC>(h + (size_t)t * C + c, u[i]);
+            } else {
+#pragma unroll
+                for (int v = 0; v < VEC; ++v) u[i][v] = 0.f;
+            }
+        }
+#pragma unroll
+    for (int i = 0; i < RUN; ++i) {
+        const int t = t0 + i;
+        if (t >= T || !ZLM_CHK(token_seq + t, 4)) break;
+        const int r = token_seq[t];
+        if (!ZLM_CHK(cu_seqlens + r, 8)) break;
+        const int row0 = cu_seqlens[r], at = t - row0;
+        if (at == 0) {
+            const int n = cu_seqlens[r + 1] - row0;
+            TA* st = nullptr;
+            if (taps > 1) {
+                if (!ZLM_CHK(seq_slot + r, 4)) continue;
+                st = state + (size_t)seq_slot[r] * (taps - 1) * C + c;
+                if (!ZLM_CHK(st, ((size_t)(taps - 2) * C + VEC) * sizeof(TA))) continue;
+            }
+            input_conv_head<TA, VEC>(out, h, w, st, row0, n, max(1, min(n, taps - 1)), C, c, taps);
+            continue;
+        }
+        if (at < taps - 1) continue;
+        float a[VEC];
+#pragma unroll
+        for (int v = 0; v < VEC; ++v) a[v] = 0.f;
+        if (TAPS > 0) {
+#pragma unroll
+            for (int j = 0; j < TAPS; ++j)
+#pragma unroll
+                for (int v = 0; v < VEC; ++v) a[v] = fmaf(k[j][v], u[i + j][v], a[v]);
+#pragma unroll
+            for (int v = 0; v < VEC; ++v) a[v] += u[i + TAPS - 1][v];
+        } else {
+            float x[VEC], kk[VEC];
+#pragma unroll
+            for (int v = 0; v < VEC; ++v) x[v] = 0.f;
+            for (int j = 0; j < taps; ++j) {
+                const TA* up = h + (size_t)(t - (taps - 1) + j) * C + c;
+                if (!ZLM_CHK(up, VEC * sizeof(TA))) continue;
+                load_vec<TA, VEC>(up, x);
+                load_vec<TA, VEC>(w + (size_t)j * C + c, kk);
+#pragma unroll
+                for (int v = 0; v < VEC; ++v) a[v] = fmaf(kk[v], x[v], a[v]);
+            }
+#pragma unroll
+            for (int v = 0; v < VEC; ++v) a[v] += x[v];
+        }
+        TA* o = out + (size_t)t * C + c;
+        if (ZLM_CHK(o, VEC * sizeof(TA))) store_vec<TA, VEC>(o, a);
+    }
+}
+
 template <typename TA>
 static void launch_input_conv(void* out, const void* h, const void* w, void* state, const int* token_seq, const int* cu_seqlens,
                               const int* seq_slot, int T, int C, int taps, cudaStream_t st) {
     const size_t quad = 4 * sizeof(TA);
     const bool vec = C % 4 == 0 && (uintptr_t)out % quad == 0 && (uintptr_t)h % quad == 0 && (uintptr_t)w % quad == 0 &&
                      (uintptr_t)state % quad == 0;
-    if (vec)
-        zlm_launch(input_conv_kernel<TA, 4>, dim3(T, (C / 4 + 127) / 128), dim3(128), 0, st, (TA*)out, (const TA*)h, (const TA*)w,
-                   (TA*)state, token_seq, cu_seqlens, seq_slot, C, taps);
-    else
-        zlm_launch(input_conv_kernel<TA, 1>, dim3(T, (C + 127) / 128), dim3(128), 0, st, (TA*)out, (const TA*)h, (const TA*)w,
-                   (TA*)state, token_seq, cu_seqlens, seq_slot, C, taps);
+    // runs of eight tokens share most of the rows they read; few tokens (among them steps of one token a sequence, where
+    // every token is a sequence's first) take a block each
+#define ZLM_IC(VEC, TAPS, RUN)                                                                                              \
+    zlm_launch(input_conv_kernel<TA, VEC, TAPS, RUN>, dim3((T + RUN - 1) / RUN, (C + 128 * VEC - 1) / (128 * VEC)), dim3(128), 0, st, \
+               (TA*)out, (const TA*)h, (const TA*)w, (TA*)state, token_seq, cu_seqlens, seq_slot, T, C, taps)
+    if (!vec) ZLM_IC(1, 0, 1);
+    else if (T < 512) ZLM_IC(4, 0, 1);
+    else if (taps == 2) ZLM_IC(4, 2, 8);
+    else if (taps == 3) ZLM_IC(4, 3, 8);
+    else if (taps == 4) ZLM_IC(4, 4, 8);
+    else ZLM_IC(4, 0, 8);
+#undef ZLM_IC
 }
 
 extern "C" int zlm_input_conv(void* out, const void* h, const void* w, void* state, int dtype, const int* token_seq,

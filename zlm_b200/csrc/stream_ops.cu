@@ -184,11 +184,12 @@ extern "C" int zlm_norm_scale_add(float* stream, const void* y, int y_dtype, con
 // stream += y / rms(y) * w1, then out2 = norm(stream) * w2 in the element type: a layer that norms a sublayer's
 // output and the next sublayer's input does both in one pass over the row, which is held in registers (or, where it does
 // not fit them, in shared memory) as fp32.  norm is x / rms(x), or with CENTER d / rms(d), d = x - mean(x) (layer norm).
-// One block per row, its size a function of H alone.
+// One block per row, its size a function of H and of whether the rows are few.
 //
 // `tail` (steps of one token a sequence; taps 0: none): the next layer's causal convolution over time of the rows just
 // normed, mixed[r] = h + sum_j w[j] * u_j with u the taps - 1 rows before (the slot's state, oldest first) and h itself
 // last; the state then takes h in.  h is the row as out2 holds it.
+#define NAN_FEW_ROWS 128
 struct ConvTail {
     const void* w;              // [taps][H] in the element type
     int taps;
@@ -231,21 +232,35 @@ template <typename TO> __device__ __forceinline__ float4 as_stored(float4 v) {
     return make_float4(to_f32(from_f32<TO>(v.x)), to_f32(from_f32<TO>(v.y)), to_f32(from_f32<TO>(v.z)), to_f32(from_f32<TO>(v.w)));
 }
 
-template <typename TO, bool CENTER>
-__global__ void norm_add_norm_kernel(float* __restrict__ stream, const float* __restrict__ y, VecW w1, float eps1,
-                                     TO* __restrict__ out2, VecW w2, float eps2, int H, int in_regs, ConvTail tail) {
+// NV: float4s of a row a thread keeps (0: the row in shared memory).  TAPS > 0 (with NV 1): that many taps, whose weights
+// and rows of state are asked for at the start, together with the row; TAPS 0: tail.taps of them, one after the other.
+template <typename TO, bool CENTER, int NV, int TAPS>
+__global__ void __launch_bounds__(1024)
+norm_add_norm_kernel(float* __restrict__ stream, const float* __restrict__ y, VecW w1, float eps1,
+                                     TO* __restrict__ out2, VecW w2, float eps2, int H, ConvTail tail) {
     extern __shared__ float nan_row[];          // [32] reduction, then (rows that do not fit the registers) [H] the row
     float* red = nan_row;
     float* row = nan_row + 32;
     pdl_trigger();
     const int r = blockIdx.x;
+    const TO* cw = (const TO*)tail.w;
+    float4 k1[NV > 0 ? NV : 1], k2[NV > 0 ? NV : 1], ck[TAPS > 0 ? TAPS : 1], cu[TAPS > 1 ? TAPS - 1 : 1];
+    if (NV == 1) {
+        // few rows: what does not change during a step is asked for ahead of the wait
+        if ((int)threadIdx.x * 4 < H) {
+            k1[0] = w1.load4(threadIdx.x * 4);
+            k2[0] = w2.load4(threadIdx.x * 4);
+            if (TAPS > 0 && ZLM_CHK(cw, (size_t)TAPS * H * sizeof(TO)))
+#pragma unroll
+                for (int j = 0; j < TAPS; ++j) ck[j] = tail_load4(cw + (size_t)j * H + threadIdx.x * 4);
+        }
+    }
     pdl_wait();
     float* xr = stream + (size_t)r * H;
     const float* yr = y + (size_t)r * H;
     TO* orow = out2 + (size_t)r * H;
     if (!ZLM_CHK(xr, (size_t)H * 4) || !ZLM_CHK(yr, (size_t)H * 4) || !ZLM_CHK(orow, (size_t)H * sizeof(TO))) return;
     TO *st = nullptr, *mixed = nullptr;
-    const TO* cw = (const TO*)tail.w;
     if (tail.taps > 0) {
         if (!ZLM_CHK(tail.seq_slot + r, 4)) return;
         mixed = (TO*)tail.mixed + (size_t)r * H;
@@ -254,26 +269,32 @@ __global__ void norm_add_norm_kernel(float* __restrict__ stream, const float* __
             (st && !ZLM_CHK(st, (size_t)(tail.taps - 1) * H * sizeof(TO))))
             return;
     }
-    if (in_regs) {
-        // H a multiple of 4 and up to NORM_MAX_V4 float4 a thread: the row is read once and stays in registers
+    if (NV > 0) {
+        // H a multiple of 4 and up to NV float4 a thread: the row is read once and stays in registers
         const int nv = H / 4;
-        float4 v[NORM_MAX_V4], x[NORM_MAX_V4];
+        float4 v[NV > 0 ? NV : 1], x[NV > 0 ? NV : 1];
         float s = 0.f;
 #pragma unroll
-        for (int j = 0; j < NORM_MAX_V4; ++j) {
+        for (int j = 0; j < NV; ++j) {
             const int c = threadIdx.x + j * blockDim.x;
             v[j] = c < nv ? *(const float4*)(yr + c * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
             x[j] = c < nv ? *(const float4*)(xr + c * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+        if (TAPS > 1 && (int)threadIdx.x < nv)
+#pragma unroll
+            for (int j = 0; j < TAPS - 1; ++j) cu[j] = tail_load4(st + (size_t)j * H + threadIdx.x * 4);
+#pragma unroll
+        for (int j = 0; j < NV; ++j) {
             s = fmaf(v[j].x, v[j].x, s); s = fmaf(v[j].y, v[j].y, s);
             s = fmaf(v[j].z, v[j].z, s); s = fmaf(v[j].w, v[j].w, s);
         }
         const float inv1 = 1.0f / sqrtf(block_sum(s, red) / (float)H + eps1);
         float s2 = 0.f;
 #pragma unroll
-        for (int j = 0; j < NORM_MAX_V4; ++j) {
+        for (int j = 0; j < NV; ++j) {
             const int c = threadIdx.x + j * blockDim.x;
             if (c >= nv) continue;
-            const float4 wv = w1.load4(c * 4);
+            const float4 wv = NV == 1 ? k1[0] : w1.load4(c * 4);
             float4 a = x[j];
             a.x += (v[j].x * inv1) * wv.x; a.y += (v[j].y * inv1) * wv.y;
             a.z += (v[j].z * inv1) * wv.z; a.w += (v[j].w * inv1) * wv.w;
@@ -290,8 +311,8 @@ __global__ void norm_add_norm_kernel(float* __restrict__ stream, const float* __
             const float mean = sq / (float)H;
             float q = 0.f;
 #pragma unroll
-            for (int j = 0; j < NORM_MAX_V4; ++j) {
-                if (threadIdx.x + j * blockDim.x >= nv) continue;
+            for (int j = 0; j < NV; ++j) {
+                if ((int)(threadIdx.x + j * blockDim.x) >= nv) continue;
                 v[j].x -= mean; v[j].y -= mean; v[j].z -= mean; v[j].w -= mean;
                 q = fmaf(v[j].x, v[j].x, q); q = fmaf(v[j].y, v[j].y, q); q = fmaf(v[j].z, v[j].z, q); q = fmaf(v[j].w, v[j].w, q);
             }
@@ -299,13 +320,26 @@ __global__ void norm_add_norm_kernel(float* __restrict__ stream, const float* __
         }
         const float inv2 = 1.0f / sqrtf(sq / (float)H + eps2);
 #pragma unroll
-        for (int j = 0; j < NORM_MAX_V4; ++j) {
+        for (int j = 0; j < NV; ++j) {
             const int c = threadIdx.x + j * blockDim.x;
             if (c >= nv) continue;
-            const float4 wv = w2.load4(c * 4);
+            const float4 wv = NV == 1 ? k2[0] : w2.load4(c * 4);
             const float4 h = make_float4((v[j].x * inv2) * wv.x, (v[j].y * inv2) * wv.y, (v[j].z * inv2) * wv.z, (v[j].w * inv2) * wv.w);
             store4(orow + c * 4, h.x, h.y, h.z, h.w);
-            if (tail.taps > 0) conv_tail_channels4<TO>(cw, st, mixed, tail.taps, H, c * 4, as_stored<TO>(h));
+            if (TAPS > 0) {
+                const float4 hs = as_stored<TO>(h);
+                float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+                for (int t = 0; t < TAPS; ++t) {
+                    const float4 u = t < TAPS - 1 ? cu[t < TAPS - 1 ? t : 0] : hs;
+                    a.x = fmaf(ck[t].x, u.x, a.x); a.y = fmaf(ck[t].y, u.y, a.y);
+                    a.z = fmaf(ck[t].z, u.z, a.z); a.w = fmaf(ck[t].w, u.w, a.w);
+                    if (t > 0) store4(st + (size_t)(t - 1) * H + c * 4, u.x, u.y, u.z, u.w);
+                }
+                store4(mixed + c * 4, hs.x + a.x, hs.y + a.y, hs.z + a.z, hs.w + a.w);
+            } else if (tail.taps > 0) {
+                conv_tail_channels4<TO>(cw, st, mixed, tail.taps, H, c * 4, as_stored<TO>(h));
+            }
         }
         return;
     }
@@ -341,13 +375,30 @@ __global__ void norm_add_norm_kernel(float* __restrict__ stream, const float* __
     }
 }
 
-template <typename TO>
-static void launch_norm_add_norm(int R, int threads, size_t smem, cudaStream_t st, float* stream, const float* y, VecW v1,
-                                 float eps1, void* out2, VecW v2, float eps2, int H, int in_regs, int center, ConvTail tail) {
-    if (center)
-        zlm_launch(norm_add_norm_kernel<TO, true>, R, threads, smem, st, stream, y, v1, eps1, (TO*)out2, v2, eps2, H, in_regs, tail);
+template <typename TO, bool CENTER>
+static void launch_norm_add_norm(int R, cudaStream_t st, float* stream, const float* y, VecW v1, float eps1, void* out2, VecW v2,
+                                 float eps2, int H, bool even, ConvTail tail) {
+    int threads = 128;
+    if (even && R <= NAN_FEW_ROWS && H <= 4096) {
+        // few rows: the whole latency of one row counts, so a thread has one float4 of it
+        while (threads * 4 < H) threads *= 2;
+#define ZLM_NAN(TAPS)                                                                                                        \
+        zlm_launch(norm_add_norm_kernel<TO, CENTER, 1, TAPS>, R, threads, 32 * sizeof(float), st, stream, y, v1, eps1, (TO*)out2, v2, \
+                   eps2, H, tail)
+        if (tail.taps == 2) ZLM_NAN(2);
+        else if (tail.taps == 3) ZLM_NAN(3);
+        else if (tail.taps == 4) ZLM_NAN(4);
+        else ZLM_NAN(0);
+#undef ZLM_NAN
+        return;
+    }
+    while (threads < 1024 && threads * 4 * NORM_MAX_V4 < H) threads *= 2;
+    if (even && H <= threads * 4 * NORM_MAX_V4)
+        zlm_launch(norm_add_norm_kernel<TO, CENTER, NORM_MAX_V4, 0>, R, threads, 32 * sizeof(float), st, stream, y, v1, eps1, (TO*)out2,
+                   v2, eps2, H, tail);
     else
-        zlm_launch(norm_add_norm_kernel<TO, false>, R, threads, smem, st, stream, y, v1, eps1, (TO*)out2, v2, eps2, H, in_regs, tail);
+        zlm_launch(norm_add_norm_kernel<TO, CENTER, 0, 0>, R, threads, (32 + (size_t)H) * sizeof(float), st, stream, y, v1, eps1,
+                   (TO*)out2, v2, eps2, H, tail);
 }
 
 // center 1: the second norm is a layer norm.  taps 0: no convolution (conv_w, state, seq_slot and mixed are not used).
@@ -358,20 +409,20 @@ extern "C" int zlm_norm_add_norm(float* stream, const float* y, const void* w1, 
     ZLM_REQUIRE(R > 0 && H > 0 && H <= 11264, "norm_add_norm: bad sizes R=%d H=%d (rows of up to 11264)", R, H);
     ZLM_REQUIRE(taps >= 0 && (taps == 0 || (conv_w && mixed && seq_slot && (taps == 1 || state))),
                 "norm_add_norm: a convolution of %d taps needs its weights, the slots' state and a place for its rows", taps);
-    int threads = 128;
-    while (threads < 1024 && threads * 4 * NORM_MAX_V4 < H) threads *= 2;
-    const int in_regs = (H % 4 == 0 && H / 4 <= NORM_MAX_V4 * threads && (uintptr_t)stream % 16 == 0 && (uintptr_t)y % 16 == 0 &&
-                         (uintptr_t)w1 % 16 == 0 && (uintptr_t)w2 % 16 == 0 && (uintptr_t)out2 % 16 == 0 &&
-                         (uintptr_t)conv_w % 16 == 0 && (uintptr_t)state % 16 == 0 && (uintptr_t)mixed % 16 == 0) ? 1 : 0;
-    const size_t smem = (size_t)(32 + (in_regs ? 0 : H)) * sizeof(float);
+    const bool even = H % 4 == 0 && (uintptr_t)stream % 16 == 0 && (uintptr_t)y % 16 == 0 && (uintptr_t)w1 % 16 == 0 &&
+                      (uintptr_t)w2 % 16 == 0 && (uintptr_t)out2 % 16 == 0 && (uintptr_t)conv_w % 16 == 0 &&
+                      (uintptr_t)state % 16 == 0 && (uintptr_t)mixed % 16 == 0;
     const VecW v1{w1, w1_dtype}, v2{w2, w2_dtype};
     const ConvTail tail{conv_w, taps, state, seq_slot, mixed};
-    if (out2_dtype == ZLM_DTYPE_F32)
-        launch_norm_add_norm<float>(R, threads, smem, st, stream, y, v1, eps1, out2, v2, eps2, H, in_regs, center, tail);
-    else if (out2_dtype == ZLM_DTYPE_BF16)
-        launch_norm_add_norm<__nv_bfloat16>(R, threads, smem, st, stream, y, v1, eps1, out2, v2, eps2, H, in_regs, center, tail);
-    else
-        ZLM_REQUIRE(false, "norm_add_norm: unsupported output dtype %d", out2_dtype);
+#define ZLM_NAN(TO)                                                                                                     \
+    do {                                                                                                                \
+        if (center) launch_norm_add_norm<TO, true>(R, st, stream, y, v1, eps1, out2, v2, eps2, H, even, tail);           \
+        else launch_norm_add_norm<TO, false>(R, st, stream, y, v1, eps1, out2, v2, eps2, H, even, tail);                 \
+    } while (0)
+    if (out2_dtype == ZLM_DTYPE_F32) ZLM_NAN(float);
+    else if (out2_dtype == ZLM_DTYPE_BF16) ZLM_NAN(__nv_bfloat16);
+    else ZLM_REQUIRE(false, "norm_add_norm: unsupported output dtype %d", out2_dtype);
+#undef ZLM_NAN
     return zlm_check_launch("norm_add_norm");
 }
 

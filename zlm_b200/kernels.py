@@ -7,6 +7,7 @@ library or without a GPU raises.
 """
 from __future__ import annotations
 
+import contextlib
 import ctypes
 from ctypes import c_float, c_int, c_void_p
 from typing import Optional
@@ -180,6 +181,9 @@ class CudaKernels:
         self._lazy_ok = False          # the next norm's output is read by products only (the arrangement's word)
         self._lazy = None              # (out, stream, weight, eps, rows times weight, sums of squares, blocks): a norm not run
         self._blank = None             # a tensor that is to be taken as zeros (see expect_blank)
+        self._lane = 0                 # 1 while calls go to the side stream (see side_lane)
+        self._side = None
+        self._join = None              # (tensor, event): who touches the tensor next waits for the event first
         self.gated_activations = ("silu", "gelu_tanh", "swish_limit")      # what linear_swiglu's ``act`` takes
         self._scratch = {}
         self.scratch_generation = 0
@@ -189,6 +193,8 @@ class CudaKernels:
         """Scratch memory that a kernel needs beyond its operands.  It grows when asked for
         more and keeps its address otherwise; ``scratch_generation`` counts the moves, so
         that a captured graph that holds an old address is not replayed."""
+        if self._lane:
+            name += "/side"             # (what runs on the other stream at the same time has scratch of its own)
         buf = self._scratch.get(name)
         if buf is None or buf.numel() < n or buf.dtype != dtype or buf.device != device:
             self._scratch[name] = buf = torch.empty(max(n, 1 << 16), dtype=dtype, device=device)
@@ -221,6 +227,8 @@ class CudaKernels:
         spans are also noted as memory the next call may touch."""
         if t is None:
             return c_void_p(0)
+        if self._join is not None and self._overlap(t, self._join[0]):
+            self.join()
         if self._shares is not None:
             # a product whose shares of K are not added up yet: whoever touches its output gets it finished first
             lo, n = self._shares[0].data_ptr(), _span_bytes(self._shares[0])
@@ -272,10 +280,41 @@ class CudaKernels:
         before the reading part writes into the stream, and by nobody after that.  Holds for one call."""
         self._lazy_ok = bool(yes) and self.lazy_norms
 
+    @contextlib.contextmanager
+    def side_lane(self, shared: torch.Tensor):
+        """Kernels launched inside the block go to a second stream of high priority, which starts when everything queued
+        so far is done; what is queued after the block runs beside them.  ``shared`` is the tensor that both sides add
+        into: the first call that is given it afterwards has its stream wait for the side stream (``join`` does so at any
+        time; the caller makes sure that one of the two happens).  The two sides may share nothing else that either
+        writes; scratch that this class hands out is kept apart."""
+        main = torch.cuda.current_stream()
+        if self._side is None or self._side.device != main.device:
+            self._side = torch.cuda.Stream(device=main.device, priority=-1)
+        self.join()
+        self.flush_shares()
+        self._side.wait_stream(main)
+        self._lane = 1
+        try:
+            with torch.cuda.stream(self._side):
+                yield
+                self.flush_shares()
+                done = torch.cuda.Event()
+                done.record()
+        finally:
+            self._lane = 0
+        self._join = (shared, done)
+
+    def join(self) -> None:
+        """Has the current stream wait for what ``side_lane`` queued, if it has not yet."""
+        if self._join is not None:
+            (_, done), self._join = self._join, None
+            torch.cuda.current_stream().wait_event(done)
+
     def forget_pending(self) -> None:
         """Drops what one call left for a later one (shares of K, a norm's halves, a norm not run, the
         arrangement's words) without finishing any of it: for the start of a step, where anything still
         pending belongs to a step that was given up."""
+        self.join()
         self._shares = self._norm_hint = self._norm_halves = self._lazy = self._blank = None
         self._lazy_ok = False
 
@@ -957,28 +996,24 @@ class CudaKernels:
         call(2)
 
     def mingru(self, out: torch.Tensor, proj: torch.Tensor, z_off: int, x_off: int, g_off: int, bz: Optional[torch.Tensor],
-               bx: Optional[torch.Tensor], state: torch.Tensor, plan, pieces: Optional[bool] = None) -> None:
+               bx: Optional[torch.Tensor], state: torch.Tensor, plan, cluster: Optional[bool] = None) -> None:
         """out[t] = S_t silu(g), S_t = (1 - z) S_(t-1) + z cand, z = sigmoid(zp + bz), cand = u + 1/2 where u = xp + bx >= 0
         and sigmoid(u) elsewhere; zp, xp and g are the W columns of ``proj`` from z_off, x_off and g_off on, ``state``
-        [slots, W] fp32.  Long prompts run in pieces side by side (``pieces`` forces or forbids that)."""
+        [slots, W] fp32.  Long prompts run on clusters of blocks that share a sequence's tokens
+        (``cluster`` forces or forbids that)."""
         T = proj.shape[0]
         W = state.shape[1]
         assert out.shape == (T, W) and out.dtype == proj.dtype and out.stride(1) == 1 and proj.stride(1) == 1
         assert state.dtype == torch.float32 and state.dim() == 2 and state.is_contiguous()
         for b in (bz, bx):
             assert b is None or (b.shape == (W,) and b.is_contiguous() and b.dtype == (bz if bz is not None else bx).dtype)
-        max_new = int(getattr(plan, "max_new", 0) or 0)
-        if pieces is None:
-            pieces = max_new >= self.RECURRENT_PIECES_FROM
-        part = None
-        if pieces:
-            maxp = (max_new + self.RECURRENT_PIECE - 1) // self.RECURRENT_PIECE
-            part = plan.scratch("mingru.pieces", (2 * plan.R * maxp * W,), torch.float32)
+        if cluster is None:
+            cluster = int(getattr(plan, "max_new", 0) or 0) >= self.RECURRENT_PIECES_FROM
         b = bz if bz is not None else bx
         self._call("zlm_mingru", self._p(out), c_int(out.stride(0)), self._p(proj), c_int(proj.stride(0)), c_int(z_off),
                    c_int(x_off), c_int(g_off), self._p(bz), self._p(bx), c_int(_dt(b) if b is not None else F32), self._p(state),
                    c_int(_dt(proj)), self._p(plan.seq_slot), self._p(plan.cu_seqlens), c_int(T), c_int(plan.R), c_int(W),
-                   c_int(max_new), self._p(part), self._stream())
+                   c_int(1 if cluster else 0), self._stream())
 
     def lowrank_decay(self, alpha: torch.Tensor, proj: torch.Tensor, lo_off: int, w2: torch.Tensor, b: Optional[torch.Tensor],
                       tau: float) -> None:

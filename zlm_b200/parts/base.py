@@ -102,6 +102,8 @@ class Workspace:
         key = f"{name}:{dtype}"
         buf = self._bufs.get(key)
         if buf is None or buf.numel() < n:
+            if buf is not None and buf.is_cuda and not torch.cuda.is_current_stream_capturing():
+                torch.cuda.synchronize(buf.device)      # (kernels of another stream may still be at the old memory)
             buf = torch.empty(max(n, 1), dtype=dtype, device=self.device)
             self._bufs[key] = buf
             self.generation += 1

@@ -221,9 +221,12 @@ class SandwichNormBlock(Part):
 class ParallelSublayersBlock(Part):
     """x <- x + (mixer(m) + ffn(n)) with n = norm(x) and m = n, or what ``mixer_input`` makes of n; then ``layer_input``.
 
-    Both sublayers add their results into the stream themselves.  A layer input ends with a norm whose result is added to
+    Both sublayers add their results into the stream themselves.  In steps of one token a sequence they run at the same time,
+    on two streams, up to the products that add (``side_by_side`` False: one after the other).  A layer input ends with a norm whose result is added to
     the stream; where a block of this arrangement follows, that kernel also leaves the next block's n and, in steps of one
     token a sequence, its m.  ``LayerIO.state`` is (the mixer's state, the mixer input's state) if either has any."""
+
+    side_by_side = True
 
     def __init__(self, hidden_size: int, mixer: Mixer, feed_forward: FeedForward, mixer_norm: Norm, feed_forward_norm: Norm,
                  mixer_input: Optional[Part] = None, layer_input: Optional[Part] = None):
@@ -279,9 +282,20 @@ class ParallelSublayersBlock(Part):
             m = rt.ws.get("block.mixed", hidden.shape, rt.dtype)
             if mixed_by != (m.data_ptr(), id(self.mixer_input)):
                 self.mixer_input.forward(m, n, ctx, input_state)
-        self.mixer.forward(m, hidden, ctx, LayerIO(cache=io.cache, state=mixer_state))
-        if not getattr(self.ffn, "is_identity", False):
+        mixer_io = LayerIO(cache=io.cache, state=mixer_state)
+        has_ffn = not getattr(self.ffn, "is_identity", False)
+        lane = getattr(k, "side_lane", None) if has_ffn and ctx.is_decode and self.side_by_side else None
+        if lane is not None:
+            # one token a sequence: the mixer is a chain of short kernels, each waiting for the one before it, and the
+            # feed-forward streams weights; neither reads what the other writes until both have their result
+            with lane(hidden):
+                self.mixer.forward(m, hidden, ctx, mixer_io)
             self.ffn.forward(n, hidden, ctx)
+            k.join()
+        else:
+            self.mixer.forward(m, hidden, ctx, mixer_io)
+            if has_ffn:
+                self.ffn.forward(n, hidden, ctx)
         if self.layer_input is not None:
             self._close(hidden, ctx, n)
 
