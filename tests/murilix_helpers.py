@@ -84,6 +84,9 @@ MURI_D = model([
     layer(lat(2, 16, 16, 16, 32, 32, 0.5, rot=(1000.0, 16), window=20), moe(16, 4, 1)),
 ], vocab=96, width=48, taps=5, side=8, scale=2.0)
 MURI = {"A": MURI_A, "B": MURI_B, "C": MURI_C, "D": MURI_D}
+# the same with a small embedding scale: with a tied head a model whose stream is mostly its token's row only ever repeats
+# that token, and says little about greedy generation
+TALKATIVE = {n: dict(copy.deepcopy(c), embedding={"scale": 0.1 if n == "C" else 0.2}) for n, c in MURI.items()}
 
 
 def make_tensors(cfg_dict, seed: int) -> Dict[str, torch.Tensor]:
@@ -127,9 +130,9 @@ def write_model(tmp_path, cfg, tensors, tag: str):
     return folder
 
 
-def make_model(tmp_path, name: str, seed: int = 0):
+def make_model(tmp_path, name: str, seed: int = 0, talkative: bool = False):
     """Writes the model to a folder; returns (folder, config mapping, float64 tensors for the oracle)."""
-    cfg = MURI[name]
+    cfg = (TALKATIVE if talkative else MURI)[name]
     tensors = make_tensors(cfg, seed)
     return write_model(tmp_path, cfg, tensors, f"{name}_{seed}"), cfg, {n: t.double() for n, t in tensors.items()}
 

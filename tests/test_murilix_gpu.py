@@ -13,9 +13,9 @@ DTYPES = ["float32", "bfloat16"]
 NAMES = sorted(MURI)
 
 
-def build(tmp_path, name, dtype, max_tokens=2048, **kw):
+def build(tmp_path, name, dtype, max_tokens=2048, talkative=False, **kw):
     from zlm_b200 import Engine
-    folder, cfg, ref = make_model(tmp_path, name, seed=5)
+    folder, cfg, ref = make_model(tmp_path, name, seed=5, talkative=talkative)
     return Engine.from_pretrained(folder, dtype=dtype, max_tokens=max_tokens, **kw), cfg, ref
 
 
@@ -131,14 +131,15 @@ def test_greedy_generation(tmp_path, name, dtype):
     """``Engine.generate`` (scheduler, decode graphs with the per-slot states inside them, sampler) against the
     oracle's greedy continuation.  32-bit: the same tokens.  bfloat16: every chosen token is, for the oracle given the
     engine's own tokens so far, the best one or within rounding of it."""
-    eng, cfg, ref = build(tmp_path, name, dtype)
+    eng, cfg, ref = build(tmp_path, name, dtype, talkative=True)
     ps = prompts(cfg["vocab"], [5, 40, 1, 66], seed=60)
     n = 12
     out = eng.generate(ps, max_tokens=n).tokens
     assert [len(o) for o in out] == [n] * len(ps)
     for p, o in zip(ps, out):
         if dtype == "float32":
-            assert o == greedy_generate(ref, cfg, p, n)
+            want = greedy_generate(ref, cfg, p, n)
+            assert o == want and len(set(want)) >= 3, f"{name}: {o} vs {want}"
         else:
             full = oracle(ref, cfg, list(p) + list(o), dtype)          # (positions that hang on a router's close call are left out)
             lg, safe = full.logits[len(p) - 1:-1], full.safe[len(p) - 1:-1]
@@ -197,7 +198,7 @@ def test_command_line_writes_and_runs_a_random_model(tmp_path, capsys):
 def test_a_batch_of_many_requests_through_captured_steps(tmp_path, name):
     """24 unequal requests generated together (decode steps of more than 16 rows: the many-token forms of the kernels
     inside captured steps) give, in 32-bit, the tokens that each request gives alone."""
-    eng, cfg, _ = build(tmp_path, name, "float32", max_tokens=64 * 64, max_batch=32)
+    eng, cfg, _ = build(tmp_path, name, "float32", max_tokens=64 * 64, max_batch=32, talkative=True)
     ps = prompts(cfg["vocab"], [3 + (7 * i) % 40 for i in range(24)], seed=9)
     together = eng.generate(ps, max_tokens=10).tokens
     alone = [eng.generate([p], max_tokens=10).tokens[0] for p in ps]

@@ -375,7 +375,8 @@ class CudaKernels:
 
     @staticmethod
     def _stream() -> c_void_p:
-        return c_void_p(torch.cuda.current_stream().cuda_stream)
+        # (the handle alone: a Stream object for every launch would cost as much host time as the rest of a call)
+        return c_void_p(torch._C._cuda_getCurrentRawStream(torch._C._cuda_getDevice()))
 
     def check_linear(self, what: str, w: torch.Tensor) -> None:
         """Raises at once, with the weight's name, if no kernel takes a product with this

@@ -250,6 +250,12 @@ class LatentAttention(Mixer):
         if made is None:
             from ..kernels import PAGE_TOKENS
             need = [(n + PAGE_TOKENS - 1) // PAGE_TOKENS for n in ctx.h_seq_new]
+            if ctx.R == 1:
+                # (made on the device: a copy from the host would have the host wait for the stream)
+                made = (torch.arange(need[0], dtype=torch.int32, device=self.rt.device).view(1, -1),
+                        torch.zeros(1, dtype=torch.int32, device=self.rt.device), need[0])
+                ctx.extras["latent.step_pages"] = made
+                return made
             table = torch.zeros((ctx.R, max(need)), dtype=torch.int32)
             at = 0
             for i, n in enumerate(need):
