@@ -80,10 +80,12 @@ __device__ __forceinline__ void route_choose(float* sc, float* cs, float* gm, in
         // every lane adds its share, then the lanes' sums meet in a butterfly: the same bits in every lane, in an
         // order that depends on E alone
         float part = 0.f;
-        for (int e = lane; e < E; e += 32) part += expf(sc[e] - mx);
+        for (int e = lane; e < E; e += 32) {            // (a lane's own scores: nobody else reads them before the sync)
+            sc[e] = expf(sc[e] - mx);
+            part += sc[e];
+        }
         const float sum = warp_sum(part);
-        __syncwarp();
-        for (int e = lane; e < E; e += 32) sc[e] = expf(sc[e] - mx) / sum;
+        for (int e = lane; e < E; e += 32) sc[e] /= sum;
         __syncwarp();
     }
     for (int e = lane; e < E; e += 32) cs[e] = sc[e] + ((corr && ZLM_CHK(corr + e, 4)) ? corr[e] : 0.f);
@@ -110,23 +112,31 @@ __device__ __forceinline__ void route_choose(float* sc, float* cs, float* gm, in
             if (gm[e / size] != -INFINITY) cs[e] = -INFINITY;       // not among the best groups
         __syncwarp();
     }
-    float chosen_sum = 0.f;
+    float chosen_sum = 0.f, my_w = 0.f;
+    int my_e = 0;                               // up to 32 choices: lane j keeps the j-th and writes it once, at the end
     for (int j = 0; j < top; ++j) {
         float bv;
         int bi;
         warp_argmax(cs, E, lane, bv, bi);
         if (bi >= E) bi = 0;                                        // (fewer candidates than top: refused by the host)
         const float s = sc[bi];
-        if (lane == 0 && ZLM_CHK(idx + (size_t)t * top + j, 4) && ZLM_CHK(wgt + (size_t)t * top + j, 4)) {
+        if (lane == j) { my_w = s * wscale; my_e = bi; }
+        if (lane == 0) cs[bi] = -INFINITY;
+        if (top > 32 && lane == 0 && ZLM_CHK(idx + (size_t)t * top + j, 4) && ZLM_CHK(wgt + (size_t)t * top + j, 4)) {
             idx[(size_t)t * top + j] = bi;
             wgt[(size_t)t * top + j] = s * wscale;
-            cs[bi] = -INFINITY;
         }
         chosen_sum += s;
         __syncwarp();
     }
-    if (renorm && lane == 0)
+    if (top <= 32) {
+        if (lane < top && ZLM_CHK(idx + (size_t)t * top + lane, 4) && ZLM_CHK(wgt + (size_t)t * top + lane, 4)) {
+            idx[(size_t)t * top + lane] = my_e;
+            wgt[(size_t)t * top + lane] = renorm ? my_w / chosen_sum : my_w;
+        }
+    } else if (renorm && lane == 0) {
         for (int j = 0; j < top; ++j) wgt[(size_t)t * top + j] /= chosen_sum;
+    }
 }
 
 #define ROUTE_WARPS 32
