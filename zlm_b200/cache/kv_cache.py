@@ -87,11 +87,11 @@ class CacheGroup:
 
     def __init__(self, request: CacheRequest, entries: List[int], num_pages: int, num_slots: int,
                  max_pages_per_slot: int, dtype: torch.dtype, device, stager: Optional[TableStager] = None,
-                 reach: Sequence[Tuple[int, int]] = ()):
-        """``reach``: (window, chunk) of every entry that reads this group's cache, its own entries among them (empty:
+                 reach: Sequence[Tuple[int, int, int]] = ()):
+        """``reach``: (window, chunk, first keys kept) of every entry that reads this group's cache, its own entries among them (empty:
         the request's)."""
         self.request = request
-        self.reach = tuple(reach) or ((request.window, request.chunk),)
+        self.reach = tuple(reach) or ((request.window, request.chunk, request.keep),)
         self.stager = stager
         self.entries = entries
         self.num_pages = num_pages
@@ -133,16 +133,18 @@ class CacheGroup:
     def trim(self, slot: int, length: int) -> None:
         """Window and chunk groups: give back the pages whose keys can no longer be read by any entry.
         The next query sits at position ``length`` and reads keys >= length + 1 - window, and with
-        chunks none before the start of its own chunk."""
+        chunks none before the start of its own chunk; beside a window it may read the sequence's first keys, whose
+        pages are kept."""
         def first(window: int, chunk: int) -> int:
             lo = max(0, length + 1 - window) if window else 0
             return max(lo, length - length % chunk) if chunk else lo
-        first_needed = min(first(w, c) for w, c in self.reach)
+        first_needed = min(first(w, c) for w, c, _ in self.reach)
+        kept = pages_for(max(k for _, _, k in self.reach))
         if first_needed < PAGE_TOKENS:
             return
         have = self.slot_pages.get(slot, [])
         back = []
-        for lp in range(min(len(have), first_needed // PAGE_TOKENS)):
+        for lp in range(kept, min(len(have), first_needed // PAGE_TOKENS)):
             if have[lp] >= 0:
                 back.append(have[lp])
                 have[lp] = -1
@@ -183,7 +185,7 @@ class KVCache:
         readers: Dict[int, set] = {}
         for i, (e, r) in enumerate(zip(schedule, requests)):
             if r is not None:
-                readers.setdefault(i if e.cache_of is None else e.cache_of, set()).add((r.window, r.chunk))
+                readers.setdefault(i if e.cache_of is None else e.cache_of, set()).add((r.window, r.chunk, r.keep))
         by_req: Dict[Tuple, List[int]] = {}
         for i, (e, r) in enumerate(zip(schedule, requests)):
             if r is not None and e.cache_of is None:

@@ -4,7 +4,8 @@ from .nuvilorn import NuvilornConfig
 from .zekazen import ZekazenConfig
 from .lodevik import LodevikConfig
 from .sudupel import SudupelConfig
+from .lolivik import LolivikConfig
 from .murilix import MurilixConfig
 
 __all__ = ["ConfigError", "LayerSpec", "ModelSpec", "PartSpec", "ScheduleEntry", "Qwen3Config", "NuvilornConfig",
-           "ZekazenConfig", "LodevikConfig", "SudupelConfig", "MurilixConfig"]
+           "ZekazenConfig", "LodevikConfig", "SudupelConfig", "MurilixConfig", "LolivikConfig"]

@@ -35,13 +35,13 @@ attention_decode_kernel(__nv_bfloat16* __restrict__ out, int out_stride, const _
 __global__ void __launch_bounds__(COMB_THREADS)
 attention_decode_combine_kernel(__nv_bfloat16* __restrict__ out, int out_stride, const float* __restrict__ part_o,
                                 const float* __restrict__ part_ml, const int* __restrict__ token_pos, int nq,
-                                int hd, int splits, int per, int window, int chunk) {
+                                int hd, int splits, int per, int window, int chunk, int keep) {
     __shared__ float fs[COMB_MAX_SPLITS];
     __shared__ float red[32];
     pdl_trigger();
     pdl_wait();
     attention_decode_combine_item(fs, red, threadIdx.x, GroupSync{0, COMB_THREADS}, blockIdx.x, blockIdx.y, out,
-                                  out_stride, part_o, part_ml, token_pos, nq, hd, splits, per, window, chunk);
+                                  out_stride, part_o, part_ml, token_pos, nq, hd, splits, per, window, chunk, keep);
 }
 
 template <int HD>
@@ -71,7 +71,7 @@ static int launch_decode(__nv_bfloat16* out, int out_stride, const __nv_bfloat16
     if (rc) return rc;
     if (splits > 1) {
         zlm_launch(attention_decode_combine_kernel, dim3(T, nq), dim3(COMB_THREADS), 0, st, out, out_stride,
-                   (const float*)part_o, (const float*)part_ml, token_pos, nq, HD, splits, per, window, opt.chunk);
+                   (const float*)part_o, (const float*)part_ml, token_pos, nq, HD, splits, per, window, opt.chunk, opt.keep);
         rc = zlm_check_launch("attention_decode_combine");
     }
     return rc;
@@ -87,7 +87,7 @@ extern "C" int zlm_attention_decode_combine_chunk(void* out, int out_stride, con
     ZLM_REQUIRE(splits >= 1 && splits <= COMB_MAX_SPLITS && nq > 0 && nq <= 65535 && hd > 0 && per >= 1 && chunk >= 0,
                 "attention_decode_combine: splits=%d heads=%d size=%d", splits, nq, hd);
     zlm_launch(attention_decode_combine_kernel, dim3(T, nq), dim3(COMB_THREADS), 0, st, (__nv_bfloat16*)out, out_stride,
-               part_o, part_ml, token_pos, nq, hd, splits, per, window, chunk);
+               part_o, part_ml, token_pos, nq, hd, splits, per, window, chunk, 0);
     return zlm_check_launch("attention_decode_combine");
 }
 
@@ -108,17 +108,16 @@ extern "C" int zlm_attention_decode_supported(int nq, int nkv, int hd) {
 // (1 for a decode step); pages that hold older positions only are read before the wait for the
 // kernel before this one.  0: not known, nothing is read early.
 // sink: the softmax has one more term, a key of score 0 that has no value (its denominator is 1 + sum exp(s)).
-// chunk, softcap, sinks, v_share: the options of AttnOpts (attn_common.cuh).
+// chunk, softcap, sinks, v_share, keep, bias, bias_n: the options of AttnOpts (attn_common.cuh).
 extern "C" int zlm_attention_decode_fresh(void* out, int out_stride, const void* q, int q_stride, const void* pool,
                                           const int* block_table, int table_stride, const int* token_pos,
                                           const int* token_slot, int T, int nq, int nkv, int hd, float scale,
                                           int window, int splits, int per, float* part_o, float* part_ml,
                                           int fresh, int sink, int chunk, float softcap, const float* sinks,
-                                          int v_share, cudaStream_t st) {
+                                          int v_share, int keep, const float* bias, int bias_n, cudaStream_t st) {
     if (T == 0) return ZLM_OK;
-    ZLM_REQUIRE(chunk >= 0 && softcap >= 0.f && v_share >= 1 && nkv % v_share == 0,
-                "attention_decode: chunk=%d softcap=%g v_share=%d", chunk, (double)softcap, v_share);
-    const AttnOpts opt{chunk, softcap, sinks, v_share};
+    ZLM_REQUIRE_ATTN_OPTS("attention_decode");
+    const AttnOpts opt{chunk, softcap, sinks, v_share, keep, bias, bias_n};
     ZLM_REQUIRE(zlm_attention_decode_supported(nq, nkv, hd),
                 "attention_decode: %d heads over %d kv heads of size %d is not a shape this kernel takes", nq, nkv, hd);
     ZLM_REQUIRE(splits >= 1 && splits <= COMB_MAX_SPLITS && nkv <= 65535 && per >= 1,
@@ -146,7 +145,7 @@ extern "C" int zlm_attention_decode(void* out, int out_stride, const void* q, in
                                     cudaStream_t st) {
     return zlm_attention_decode_fresh(out, out_stride, q, q_stride, pool, block_table, table_stride, token_pos,
                                       token_slot, T, nq, nkv, hd, scale, window, splits, per, part_o, part_ml, 0, 0,
-                                      0, 0.f, nullptr, 1, st);
+                                      0, 0.f, nullptr, 1, 0, nullptr, 0, st);
 }
 
 // ---------------------------------------------------------------------------

@@ -17,7 +17,7 @@ __device__ __forceinline__ void attention_decode_item(
     __nv_bfloat16* out, int out_stride, const __nv_bfloat16* q, int q_stride, const __nv_bfloat16* pool,
     const int* block_table, int table_stride, const int* token_pos, const int* token_slot, int nq, int nkv,
     float scale_log2, int window, int splits, int per, float* part_o, float* part_ml, int fresh, int sink = 0,
-    AttnOpts opt = AttnOpts{0, 0.f, nullptr, 1}) {
+    AttnOpts opt = AttnOpts{0, 0.f, nullptr, 1, 0, nullptr, 0}) {
     constexpr int KS = HD / 16;            // k-steps of Q K^T; pairs of output n-tiles of P V
     constexpr int CH = HD / 8;             // 16-byte chunks per row
     constexpr int TILE = ZLM_PAGE * HD;    // elements of one K or V page of one kv head
@@ -38,9 +38,9 @@ __device__ __forceinline__ void attention_decode_item(
     const float softcap = opt.softcap;
 
     // this split's pages
-    const int page_lo = t_start / ZLM_PAGE, page_hi = pos / ZLM_PAGE + 1;
-    const int p_begin = page_lo + split * per;
-    const int p_end = min(page_hi, p_begin + per);
+    const AttnWalk walk(t_start / ZLM_PAGE, pos / ZLM_PAGE + 1, opt.keep);
+    const int p_begin = split * per;
+    const int p_end = min(walk.n, p_begin + per);
     if (p_begin >= p_end && splits > 1) return;      // the combine kernel skips this split too
 
     // q and this step's keys and values come from the kernel before; pages that hold only positions
@@ -48,9 +48,10 @@ __device__ __forceinline__ void attention_decode_item(
     // is how many of a sequence's newest positions this step may have written (0: not known,
     // nothing is read early).
     const int old_pages = fresh > 0 ? max(0, pos + 1 - fresh) / ZLM_PAGE : 0;
-    const bool early0 = PDL && p_begin < p_end && p_begin < old_pages;
-    const bool early1 = early0 && p_begin + 1 < p_end && p_begin + 1 < old_pages;
-    auto load_page = [&](int p, int stage) {
+    const bool early0 = PDL && p_begin < p_end && walk.page(p_begin) < old_pages;
+    const bool early1 = early0 && p_begin + 1 < p_end && walk.page(p_begin + 1) < old_pages;
+    auto load_page = [&](int w, int stage) {
+        const int p = walk.page(w);
         if (!ZLM_CHK(pages + p, 4)) return;
         const __nv_bfloat16* kb = pool + (size_t)pages[p] * page_stride + (size_t)kvh * TILE;
         const __nv_bfloat16* vb = kb + v_off;
@@ -112,8 +113,8 @@ __device__ __forceinline__ void attention_decode_item(
         const int stage = (p - p_begin) & 1;
         dec_wait<1>();                       // everything but the newest group has landed: page p is there
         gs.sync();
-        const int kbase = p * ZLM_PAGE + warp * 16;
-        const bool busy = !(kbase > pos || kbase + 15 < t_start);       // warp-uniform
+        const int kbase = walk.page(p) * ZLM_PAGE + warp * 16;
+        const bool busy = !(kbase > pos || (kbase + 15 < t_start && kbase >= opt.keep));       // warp-uniform
         if (busy) {
         const __nv_bfloat16* kt = Ks + stage * TILE;
         const __nv_bfloat16* vt = Vs + stage * TILE;
@@ -136,12 +137,24 @@ __device__ __forceinline__ void attention_decode_item(
         // scale (to base-2 exponent) and mask by position
         float mx0 = -INFINITY, mx1 = -INFINITY;
         attn_scores_log2<2>(s, scale_log2, softcap);
+        if (opt.bias) {                                // (rows beyond the group hold nothing that counts)
+            const float* b0 = opt.bias + (size_t)(kvh * G + min(g, G - 1)) * opt.bias_n;
+            const float* b1 = opt.bias + (size_t)(kvh * G + min(g + 8, G - 1)) * opt.bias_n;
+#pragma unroll
+            for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+                for (int e = 0; e < 2; ++e) {
+                    const int n = pos - (kbase + nt * 8 + qd * 2 + e);
+                    s[nt][e] += attn_bias_log2(b0, n, opt.bias_n);
+                    if (G > 8) s[nt][2 + e] += attn_bias_log2(b1, n, opt.bias_n);
+                }
+        }
 #pragma unroll
         for (int nt = 0; nt < 2; ++nt)
 #pragma unroll
             for (int e = 0; e < 2; ++e) {
                 const int key = kbase + nt * 8 + qd * 2 + e;
-                const bool ok = key <= pos && key >= t_start;
+                const bool ok = attn_sees(key, pos, t_start, opt.keep);
                 s[nt][e] = ok ? s[nt][e] : -INFINITY;
                 s[nt][2 + e] = ok ? s[nt][2 + e] : -INFINITY;
                 mx0 = fmaxf(mx0, s[nt][e]);
@@ -250,11 +263,11 @@ __device__ __forceinline__ void attention_decode_item(
 __device__ __forceinline__ void attention_decode_combine_item(
     float* fs, float* red, const int tid, const GroupSync gs, const int t, const int head, __nv_bfloat16* out,
     int out_stride, const float* part_o, const float* part_ml, const int* token_pos, int nq, int hd, int splits,
-    int per, int window, int chunk = 0) {
+    int per, int window, int chunk = 0, int keep = 0) {
     if (!ZLM_CHK(token_pos + t, 4)) return;
     const int pos = token_pos[t];
     const int t_start = attn_first_key(pos, window, chunk);
-    const int pages = pos / ZLM_PAGE + 1 - t_start / ZLM_PAGE;
+    const int pages = AttnWalk(t_start / ZLM_PAGE, pos / ZLM_PAGE + 1, keep).n;
     const int used = min(splits, (pages + per - 1) / per);
     const size_t base = ((size_t)t * nq + head) * splits;
     if (!ZLM_CHK(part_ml + base * 2, (size_t)used * 8) || !ZLM_CHK(part_o + base * hd, (size_t)used * hd * 4) ||

@@ -13,8 +13,10 @@
 // `softcap` (s <- cap * tanh(s / cap) after the scale), `sinks` (one number per query head whose exponential
 // joins the softmax's denominator without a value; without the array the flag `sink` stands for a 0), and
 // `v_share` (that many neighbouring key heads read one value head: the page is [nkv key heads | nkv / v_share
-// value heads] of [ZLM_PAGE][hd] each).
+// value heads] of [ZLM_PAGE][hd] each), `keep` (with a window: the sequence's first `keep` keys stay visible) and `bias`
+// ([nq][bias_n], added after the cap by distance, the last entry for all greater distances).
 #include "common.cuh"
+#include "attn_common.cuh"
 
 #define ATT_WARPS 4
 #define ATT_MAX_PER_LANE 16   // head_dim <= 512
@@ -26,7 +28,7 @@ attention_generic_kernel(TA* __restrict__ out, int out_stride, const TA* __restr
                          const int* __restrict__ block_table, int table_stride,
                          const int* __restrict__ token_pos, const int* __restrict__ token_slot,
                          int nq, int nkv, int hd, float scale, int window, int sink, int chunk, float softcap,
-                         const float* __restrict__ sinks, int v_share) {
+                         const float* __restrict__ sinks, int v_share, int keep, const float* __restrict__ bias, int bias_n) {
     extern __shared__ float sm[];
     float* qs = sm;                         // [hd]
     float* accs = sm + hd;                  // [ATT_WARPS][hd]
@@ -62,10 +64,16 @@ attention_generic_kernel(TA* __restrict__ out, int out_stride, const TA* __restr
     for (int r = 0; r < ATT_MAX_PER_LANE; ++r) acc[r] = 0.f;
 
     const int c0 = t_start / 32, c1 = pos / 32;
-    for (int c = c0 + ((warp - c0 % ATT_WARPS + ATT_WARPS) % ATT_WARPS); c <= c1; c += ATT_WARPS) {
+    const int kept = keep > 0 ? min((keep - 1) / 32 + 1, c0) : 0;         // chunks of the first kept keys ahead of the window's
+    const float* brow = bias ? bias + (size_t)h * bias_n : nullptr;
+    for (int c = warp; c <= c1; c += ATT_WARPS) {
         // chunk c holds keys [32c, 32c+32); chunk c belongs to warp c % ATT_WARPS
+        if (c >= kept && c < c0) {                 // between the kept keys and the window: on to this warp's first chunk there
+            c = c0 + ((warp - c0 % ATT_WARPS + ATT_WARPS) % ATT_WARPS);
+            if (c > c1) break;
+        }
         const int key = c * 32 + lane;
-        const bool valid = key >= t_start && key <= pos;
+        const bool valid = attn_sees(key, pos, t_start, keep);
         if (!ZLM_CHK(pages + (c * 32) / ZLM_PAGE, 4)) continue;
         const int page = pages[(c * 32) / ZLM_PAGE];
         const TA* kbase = pool + (size_t)page * page_stride + (size_t)kvh * ZLM_PAGE * hd;
@@ -79,6 +87,7 @@ attention_generic_kernel(TA* __restrict__ out, int out_stride, const TA* __restr
             for (int e = 0; e < hd; ++e) d = fmaf(qs[e], to_f32(kr[e]), d);
             s = d * scale;
             if (softcap > 0.f) s = softcap * tanhf(s / softcap);
+            if (brow && ZLM_CHK(brow + min(pos - key, bias_n - 1), 4)) s += brow[min(pos - key, bias_n - 1)];
         }
         const float cm = warp_max(s);          // the chunk holds at least one valid key
         const float mn = fmaxf(m, cm);
@@ -90,9 +99,10 @@ attention_generic_kernel(TA* __restrict__ out, int out_stride, const TA* __restr
         for (int r = 0; r < ATT_MAX_PER_LANE; ++r) acc[r] *= alpha;
         const TA* vbase = kbase + v_off;
         const int nvalid_hi = min(31, pos - c * 32);
-        const int lo = max(0, t_start - c * 32);
+        const int lo = keep > 0 ? 0 : max(0, t_start - c * 32);
         for (int jk = lo; jk <= nvalid_hi; ++jk) {
             const float pj = __shfl_sync(0xffffffffu, p, jk);
+            if (keep > 0 && !attn_sees(c * 32 + jk, pos, t_start, keep)) continue;
             const TA* vr = vbase + (size_t)((c * 32 + jk) % ZLM_PAGE) * hd;
 #pragma unroll
             for (int r = 0; r < ATT_MAX_PER_LANE; ++r) {
@@ -134,10 +144,9 @@ extern "C" int zlm_attention_generic(void* out, int out_stride, const void* q, i
                                      int table_stride, const int* token_pos,
                                      const int* token_slot, int T, int nq, int nkv, int hd,
                                      float scale, int window, int sink, int chunk, float softcap,
-                                     const float* sinks, int v_share, cudaStream_t st) {
+                                     const float* sinks, int v_share, int keep, const float* bias, int bias_n, cudaStream_t st) {
     if (T == 0) return ZLM_OK;
-    ZLM_REQUIRE(chunk >= 0 && softcap >= 0.f && v_share >= 1 && nkv % v_share == 0,
-                "attention: chunk=%d softcap=%f, %d key heads a value head over %d key heads", chunk, softcap, v_share, nkv);
+    ZLM_REQUIRE_ATTN_OPTS("attention");
     ZLM_REQUIRE(hd > 0 && hd <= 32 * ATT_MAX_PER_LANE, "attention: head_dim=%d must be at most %d", hd,
                 32 * ATT_MAX_PER_LANE);
     ZLM_REQUIRE(nq > 0 && nkv > 0 && nq % nkv == 0, "attention: %d query heads over %d kv heads", nq, nkv);
@@ -149,12 +158,12 @@ extern "C" int zlm_attention_generic(void* out, int out_stride, const void* q, i
     if (dtype == ZLM_DTYPE_F32)
         attention_generic_kernel<float><<<grid, ATT_WARPS * 32, smem, st>>>(
             (float*)out, out_stride, (const float*)q, q_stride, (const float*)pool, block_table,
-            table_stride, token_pos, token_slot, nq, nkv, hd, scale, window, sink, chunk, softcap, sinks, v_share);
+            table_stride, token_pos, token_slot, nq, nkv, hd, scale, window, sink, chunk, softcap, sinks, v_share, keep, bias, bias_n);
     else if (dtype == ZLM_DTYPE_BF16)
         attention_generic_kernel<__nv_bfloat16><<<grid, ATT_WARPS * 32, smem, st>>>(
             (__nv_bfloat16*)out, out_stride, (const __nv_bfloat16*)q, q_stride,
             (const __nv_bfloat16*)pool, block_table, table_stride, token_pos, token_slot, nq, nkv,
-            hd, scale, window, sink, chunk, softcap, sinks, v_share);
+            hd, scale, window, sink, chunk, softcap, sinks, v_share, keep, bias, bias_n);
     else
         ZLM_REQUIRE(false, "attention: unsupported dtype %d", dtype);
     return zlm_check_launch("attention_generic");

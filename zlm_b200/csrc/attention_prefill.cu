@@ -8,7 +8,8 @@
 // prompt would.
 //
 // Options (AttnOpts, attn_common.cuh): keys of the query's own chunk of positions only, a tanh cap on the
-// scores, a sink per query head in the softmax's denominator, several key heads on one value head.
+// scores, a sink per query head in the softmax's denominator, several key heads on one value head, the sequence's first
+// keys beside a window, a bias by distance.
 //
 // Formula: s_t = (q . k_t) / sqrt(hd) for t in [t_start, pos], softmax, o = sum
 // p_t v_t (src/kernels/transformer/attention.zig:86-164); per-row bound in block
@@ -71,7 +72,10 @@ attention_prefill_kernel(__nv_bfloat16* __restrict__ out, int out_stride, const 
     // keys the block and this warp can need
     const int blk_first = start + row0, blk_last = start + row0 + rows - 1;
     const int blk_lo = attn_first_key(blk_first, window, chunk);
-    const int page_lo = blk_lo / ZLM_PAGE, page_hi = blk_last / ZLM_PAGE + 1;
+    const AttnWalk walk(blk_lo / ZLM_PAGE, blk_last / ZLM_PAGE + 1, opt.keep);
+    const int keep = opt.keep;
+    const float* brow = opt.bias ? opt.bias + (size_t)head * opt.bias_n : nullptr;
+    const float far_bias = brow ? attn_bias_log2(brow, opt.bias_n, opt.bias_n) : 0.f;
     const int w_first = start + row0 + warp * 16;
     const int w_last = min(blk_last, w_first + 15);
     const int w_lo = attn_first_key(w_first, window, chunk);
@@ -102,7 +106,8 @@ attention_prefill_kernel(__nv_bfloat16* __restrict__ out, int out_stride, const 
         if (qd == 0) l0 = l1 = 1.f;
     }
 
-    auto load_page = [&](int p, int stage) {
+    auto load_page = [&](int w, int stage) {
+        const int p = walk.page(w);
         if (!ZLM_CHK(pages + p, 4)) return;
         const __nv_bfloat16* kb = pool + (size_t)pages[p] * page_stride + (size_t)kvh * TILE;
         const __nv_bfloat16* vb = kb + v_off;
@@ -115,16 +120,16 @@ attention_prefill_kernel(__nv_bfloat16* __restrict__ out, int out_stride, const 
         }
     };
 
-    load_page(page_lo, 0);
+    load_page(0, 0);
     dec_commit();
-    for (int p = page_lo; p < page_hi; ++p) {
-        const int stage = (p - page_lo) & 1;
+    for (int p = 0; p < walk.n; ++p) {
+        const int stage = p & 1;
         dec_wait<0>();
         __syncthreads();
-        if (p + 1 < page_hi) load_page(p + 1, stage ^ 1);
+        if (p + 1 < walk.n) load_page(p + 1, stage ^ 1);
         dec_commit();
-        const int kbase = p * ZLM_PAGE;
-        if (warp_idle || kbase > w_last || kbase + ZLM_PAGE - 1 < w_lo) continue;   // warp-uniform
+        const int kbase = walk.page(p) * ZLM_PAGE;
+        if (warp_idle || kbase > w_last || (kbase + ZLM_PAGE - 1 < w_lo && kbase >= keep)) continue;   // warp-uniform
         const __nv_bfloat16* kt = Ks + stage * TILE;
         const __nv_bfloat16* vt = Vs + stage * TILE;
 
@@ -150,13 +155,24 @@ attention_prefill_kernel(__nv_bfloat16* __restrict__ out, int out_stride, const 
         const bool edge = kbase + ZLM_PAGE - 1 > w_first || kbase < w_last_lo;
         float mx0 = -INFINITY, mx1 = -INFINITY;
         attn_scores_log2<8>(s, scale_log2, softcap);
+        if (brow) {
+            const bool far = w_first - (kbase + ZLM_PAGE - 1) >= opt.bias_n - 1;        // every distance reads the table's last entry
+#pragma unroll
+            for (int nt = 0; nt < 8; ++nt)
+#pragma unroll
+                for (int e = 0; e < 2; ++e) {
+                    const int key = kbase + nt * 8 + qd * 2 + e;
+                    s[nt][e] += far ? far_bias : attn_bias_log2(brow, pos0 - key, opt.bias_n);
+                    s[nt][2 + e] += far ? far_bias : attn_bias_log2(brow, pos1 - key, opt.bias_n);
+                }
+        }
 #pragma unroll
         for (int nt = 0; nt < 8; ++nt)
 #pragma unroll
             for (int e = 0; e < 2; ++e) {
                 const int key = kbase + nt * 8 + qd * 2 + e;
-                const bool a = !edge || (key <= pos0 && key >= lo0);
-                const bool c = !edge || (key <= pos1 && key >= lo1);
+                const bool a = !edge || attn_sees(key, pos0, lo0, keep);
+                const bool c = !edge || attn_sees(key, pos1, lo1, keep);
                 s[nt][e] = (a && ok0) ? s[nt][e] : -INFINITY;
                 s[nt][2 + e] = (c && ok1) ? s[nt][2 + e] : -INFINITY;
                 mx0 = fmaxf(mx0, s[nt][e]);
@@ -265,13 +281,12 @@ extern "C" int zlm_attention_prefill(void* out, int out_stride, const void* q, i
                                      const int* block_table, int table_stride, const int* cu_seqlens,
                                      const int* seq_slot, const int* seq_start, int R, int max_new, int nq,
                                      int nkv, int hd, float scale, int window, int sink, int chunk, float softcap,
-                                     const float* sinks, int v_share, cudaStream_t st) {
+                                     const float* sinks, int v_share, int keep, const float* bias, int bias_n, cudaStream_t st) {
     if (R == 0 || max_new == 0) return ZLM_OK;
     ZLM_REQUIRE(zlm_attention_prefill_supported(nq, nkv, hd),
                 "attention_prefill: %d heads over %d kv heads of size %d is not a shape this kernel takes", nq, nkv, hd);
-    ZLM_REQUIRE(chunk >= 0 && softcap >= 0.f && v_share >= 1 && nkv % v_share == 0,
-                "attention_prefill: chunk=%d softcap=%g v_share=%d", chunk, (double)softcap, v_share);
-    const AttnOpts opt{chunk, softcap, sinks, v_share};
+    ZLM_REQUIRE_ATTN_OPTS("attention_prefill");
+    const AttnOpts opt{chunk, softcap, sinks, v_share, keep, bias, bias_n};
     ZLM_REQUIRE(q_stride % 2 == 0 && out_stride % 2 == 0 && ((uintptr_t)q % 4 == 0) && ((uintptr_t)out % 4 == 0),
                 "attention_prefill: q and out must be 4-byte aligned");
 #define ZLM_PRE_CASE(H)                                                                                         \
@@ -299,13 +314,13 @@ extern "C" int zlm_attention_prefill_vd(void* out, int out_stride, const void* q
                                         const int* block_table, int table_stride, const int* cu_seqlens,
                                         const int* seq_slot, const int* seq_start, int R, int max_new, int nq,
                                         int nkv, int hd, int vd, float scale, int window, int sink, int chunk,
-                                        float softcap, const float* sinks, int v_share, cudaStream_t st) {
+                                        float softcap, const float* sinks, int v_share, int keep, const float* bias,
+                                        int bias_n, cudaStream_t st) {
     if (R == 0 || max_new == 0) return ZLM_OK;
     ZLM_REQUIRE(zlm_attention_prefill_vd_supported(nq, nkv, hd, vd),
                 "attention_prefill: keys of %d with values of %d columns is not a pair this kernel is built for", hd, vd);
-    ZLM_REQUIRE(chunk >= 0 && softcap >= 0.f && v_share >= 1 && nkv % v_share == 0,
-                "attention_prefill: chunk=%d softcap=%g v_share=%d", chunk, (double)softcap, v_share);
-    const AttnOpts opt{chunk, softcap, sinks, v_share};
+    ZLM_REQUIRE_ATTN_OPTS("attention_prefill");
+    const AttnOpts opt{chunk, softcap, sinks, v_share, keep, bias, bias_n};
     ZLM_REQUIRE(q_stride % 2 == 0 && out_stride % 2 == 0 && ((uintptr_t)q % 4 == 0) && ((uintptr_t)out % 4 == 0),
                 "attention_prefill: q and out must be 4-byte aligned");
 #define ZLM_PRE_VD(H, V)                                                                                           \

@@ -25,7 +25,9 @@
 //
 // Options (AttnOpts, attn_common.cuh): keys of the query's own chunk of positions only; a tanh cap on the scores
 // (tanh through one exponential and one reciprocal of the special-function unit, so a capped step costs the softmax
-// warps three such operations a score instead of one); a sink per query head; several key heads on one value head.
+// warps three such operations a score instead of one); a sink per query head; several key heads on one value head; the
+// sequence's first keys beside a window; a bias by distance (heads of 128 only), read from the table where a step's
+// distances differ and added as one number where they all read its last entry.
 //
 // Formula: s_t = (q . k_t) / sqrt(hd) for t in [t_start, pos], softmax, o = sum p_t v_t
 // (src/kernels/transformer/attention.zig:86-164; per-row bound in block prefill:
@@ -121,7 +123,11 @@ __device__ __forceinline__ void fa_commit(uint64_t* bar) {
 
 // CAP: built with the cap on the scores (the form without it keeps the plain softmax's registers)
 // KD: the keys' and queries' width (128, or 192 with values of 128: rows of the pool and of q and out are KD wide)
-template <int HPC, bool CAP, int KD = FA_HD>
+// EXTRA: FA_BIAS, built with a bias by distance; FA_KEEP, with first keys kept beside the window (not both)
+#define FA_PLAIN 0
+#define FA_BIAS 1
+#define FA_KEEP 2
+template <int HPC, bool CAP, int KD = FA_HD, int EXTRA = FA_PLAIN>
 __global__ void __launch_bounds__(FA_THREADS(HPC), 1)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_kv,
                             __nv_bfloat16* __restrict__ out, int out_stride, const int* __restrict__ block_table,
@@ -187,9 +193,10 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     const int blk_lo = attn_first_key(first_pos, window, opt.chunk);
     const int last_lo = attn_first_key(last_pos, window, opt.chunk);        // (a row's first key does not fall as positions grow)
     const int page_heads = nkv + nkv / opt.v_share;                         // heads of [64][128] in a page: keys, then values
-    const int page_lo = blk_lo / ZLM_PAGE, page_hi = last_pos / ZLM_PAGE + 1;
-    const int NP = page_hi - page_lo;
-    const int NS = (NP + 1) / 2;               // steps of two pages
+    const int page_hi = last_pos / ZLM_PAGE + 1;
+    constexpr bool BIAS = EXTRA == FA_BIAS, KEEP = EXTRA == FA_KEEP;
+    const AttnWalk walk(blk_lo / ZLM_PAGE, page_hi, KEEP ? opt.keep : 0);
+    const int NS = (walk.n + 1) / 2;           // steps of two pages
 
     // K and V of step j into their stages (the producer thread; false if a wait gave up)
     int k_issued = 0, v_issued = 0;
@@ -198,7 +205,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
 #pragma unroll
         for (int pg = 0; pg < 2; ++pg) {
             // an odd last page comes twice: its second copy's keys are beyond every row's position
-            const int lp = min(page_lo + 2 * j + pg, page_hi - 1);
+            const int lp = min(walk.page(2 * j + pg), page_hi - 1);
             page[pg] = ZLM_CHK(pages + lp, 4) ? pages[lp] : 0;
         }
         const int sk = j % KST, sv = j % VST;
@@ -336,15 +343,19 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         // (sink: a key of score 0, or sinks[head], without a value, one more term in the row's sum)
         float m_ref = sink ? attn_sink_log2(opt.sinks, head) : -INFINITY, l = sink ? 1.f : 0.f;
         constexpr bool capped = CAP;
+        const int keep = KEEP ? opt.keep : 0;
+        const float* brow = BIAS ? opt.bias + (size_t)head * opt.bias_n : nullptr;
+        const float far_bias = BIAS ? attn_bias_log2(brow, opt.bias_n, opt.bias_n) : 0.f;
         const float k_in = capped ? 2.0f * scale_log2 / opt.softcap : 0.f, k_out = opt.softcap * 1.4426950408889634f;
         bool ok = true;
         for (int j = 0; j < NS; ++j) {
             ok = mbar_wait_warp(&s_full[hh], j & 1, abort_flag, 3);
             tc_fence_after();
             if (!ok || *abort_flag) { ok = false; break; }
-            const int kbase = (page_lo + 2 * j) * ZLM_PAGE;
+            // the step's two pages need not be neighbours: the kept ones lie before the window's
+            const int kb0 = (KEEP ? walk.page(2 * j) : walk.lo + 2 * j) * ZLM_PAGE, kb1 = KEEP ? walk.page(2 * j + 1) * ZLM_PAGE : kb0 + ZLM_PAGE;
             // a step that every row of the tile sees whole needs no mask (block-uniform test)
-            const bool inner = rows == FA_BM && kbase + FA_BK - 1 <= first_pos && kbase >= last_lo;
+            const bool inner = rows == FA_BM && kb1 + ZLM_PAGE - 1 <= first_pos && kb0 >= last_lo;
             // the row's 128 scores into registers in one round trip to tensor memory; then S is free
             float sv[FA_BK];
 #pragma unroll
@@ -353,7 +364,17 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             tc_fence_before();
             __syncwarp();
             if (lane == 0) mbar_arrive(&s_empty[hh]);
-            // four independent chains of maxima (raw scores; the scale is positive)
+            // a bias that differs from key to key goes into the scores before their maximum: they are then final base-2
+            // exponents; the scores of a step whose distances all read the table's last entry stay raw
+            const bool near = BIAS && first_pos - (kb1 + ZLM_PAGE - 1) < opt.bias_n - 1;        // block-uniform
+            if (near) {
+#pragma unroll
+                for (int e = 0; e < FA_BK; ++e) {
+                    const int key = kb0 + e;
+                    sv[e] = (capped ? fa_cap(sv[e], k_in, k_out) : sv[e] * scale_log2) + attn_bias_log2(brow, pos - key, opt.bias_n);
+                }
+            }
+            // four independent chains of maxima (raw scores, unless the bias went in; the scale is positive)
             float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
             if (inner) {
 #pragma unroll
@@ -361,15 +382,15 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             } else {
 #pragma unroll
                 for (int e = 0; e < FA_BK; ++e) {
-                    const int key = kbase + e;
-                    const bool vis = row_ok && key <= pos && key >= lo;
+                    const int key = (!KEEP || e < ZLM_PAGE ? kb0 : kb1 - ZLM_PAGE) + e;
+                    const bool vis = row_ok && (KEEP ? attn_sees(key, pos, lo, keep) : key <= pos && key >= lo);
                     sv[e] = vis ? sv[e] : -INFINITY;
                     mx4[e & 3] = fmaxf(mx4[e & 3], sv[e]);
                 }
             }
             // (the cap is monotonic too: the capped maximum is the maximum's cap)
             const float mx_raw = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
-            const float mx = capped ? fa_cap(mx_raw, k_in, k_out) : mx_raw * scale_log2;          // -inf stays -inf
+            const float mx = near ? mx_raw : (capped ? fa_cap(mx_raw, k_in, k_out) : mx_raw * scale_log2) + (BIAS ? far_bias : 0.f);          // -inf stays -inf
             // lazy reference: move it only when the maximum grew by more than 2^8
             const bool grow = mx > m_ref + FA_RESCALE;              // also true for the first real maximum
             const float m_new = grow ? mx : m_ref;
@@ -396,7 +417,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             }
             l *= alpha;
             m_ref = m_new;
-            const float ref = m_ref == -INFINITY ? 0.f : m_ref;
+            const float ref = (m_ref == -INFINITY ? 0.f : m_ref) - (BIAS && !near ? far_bias : 0.f);
             // P = 2^(s * scale - ref) (2^-inf = 0 for masked keys) -> shared memory: two halves of 64
             // keys, 128 bytes a row, 16-byte chunks swizzled by (row % 8)
             float ps4[4] = {0.f, 0.f, 0.f, 0.f};
@@ -405,7 +426,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                 float p[8];
 #pragma unroll
                 for (int e = 0; e < 8; ++e) {
-                    p[e] = capped ? fa_ex2(fa_cap(sv[ch * 8 + e], k_in, k_out) - ref)
+                    p[e] = near ? fa_ex2(sv[ch * 8 + e] - ref)
+                         : capped ? fa_ex2(fa_cap(sv[ch * 8 + e], k_in, k_out) - ref)
                                   : fa_ex2(fmaf(sv[ch * 8 + e], scale_log2, -ref));
                     ps4[e & 3] += p[e];
                 }
@@ -495,11 +517,11 @@ extern "C" int zlm_attention_prefill_tc_vd(void* out, int out_stride, const void
                                            int table_stride, const int* cu_seqlens, const int* seq_slot,
                                            const int* seq_start, int R, int max_new, int nq, int nkv, int hd, int vd,
                                            float scale, int window, int sink, int chunk, float softcap, const float* sinks,
-                                           int v_share, cudaStream_t st) {
+                                           int v_share, int keep, const float* bias, int bias_n, cudaStream_t st) {
     if (R == 0 || max_new == 0) return ZLM_OK;
-    ZLM_REQUIRE(chunk >= 0 && softcap >= 0.f && v_share >= 1 && nkv % v_share == 0,
-                "attention_prefill_tc: chunk=%d softcap=%g v_share=%d", chunk, (double)softcap, v_share);
-    const AttnOpts opt{chunk, softcap, sinks, v_share};
+    ZLM_REQUIRE_ATTN_OPTS("attention_prefill_tc");
+    ZLM_REQUIRE(!(bias && keep) && (hd == FA_HD || !(bias || keep)), "attention_prefill_tc: a bias by distance and kept keys are built for heads of %d, one of them at a time", FA_HD);
+    const AttnOpts opt{chunk, softcap, sinks, v_share, keep, bias, bias_n};
     const long long page_heads = nkv + nkv / v_share;
     ZLM_REQUIRE(zlm_attention_prefill_tc_vd_supported(nq, nkv, hd, vd, q_stride, out_stride),
                 "attention_prefill_tc: %d heads over %d kv heads of size %d, values of %d (strides %d, %d) is not a shape this kernel takes",
@@ -518,11 +540,11 @@ extern "C" int zlm_attention_prefill_tc_vd(void* out, int out_stride, const void
     // seven tiles of 32 KB (Q and P per head, the K and V stages), barriers, and what is left of a kilobyte for rounding the base up
     size_t smem = (size_t)7 * FA_BK * FA_HD * 2 + 256 + 1024;
     if (smem > 232448) smem = 232448;
-#define ZLM_FA_LAUNCH(H, C, KD)                                                                                    \
+#define ZLM_FA_LAUNCH(H, C, KD, B)                                                                                  \
     {                                                                                                             \
         static bool attr_set_dev[64] = {}; bool& attr_set = attr_set_dev[zlm_device_index()];                     \
         if (!attr_set) {                                                                                          \
-            cudaError_t e = cudaFuncSetAttribute(attention_prefill_tc_kernel<H, C, KD>,                              \
+            cudaError_t e = cudaFuncSetAttribute(attention_prefill_tc_kernel<H, C, KD, B>,                           \
                                                  cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);         \
             if (e != cudaSuccess) {                                                                               \
                 zlm_set_error("attention_prefill_tc: cannot reserve %zu bytes of shared memory: %s", smem,        \
@@ -531,20 +553,29 @@ extern "C" int zlm_attention_prefill_tc_vd(void* out, int out_stride, const void
             }                                                                                                     \
             attr_set = true;                                                                                      \
         }                                                                                                         \
-        zlm_launch(attention_prefill_tc_kernel<H, C, KD>, dim3(R * tiles * (nq / H)), dim3(FA_THREADS(H)), smem, st, mq, mkv, \
+        zlm_launch(attention_prefill_tc_kernel<H, C, KD, B>, dim3(R * tiles * (nq / H)), dim3(FA_THREADS(H)), smem, st, mq, mkv, \
                    (__nv_bfloat16*)out, out_stride, block_table, table_stride, cu_seqlens, seq_slot, seq_start,   \
                    R, tiles, nq, nkv, scale * 1.4426950408889634f, window, sink, opt);                                       \
     }
-    if (hd > FA_HD) {
-        if (softcap > 0.f) ZLM_FA_LAUNCH(1, true, 192)
-        else ZLM_FA_LAUNCH(1, false, 192)
-    } else if (softcap > 0.f) {
-        if (hpc == 2) ZLM_FA_LAUNCH(2, true, FA_HD)
-        else ZLM_FA_LAUNCH(1, true, FA_HD)
-    } else {
-        if (hpc == 2) ZLM_FA_LAUNCH(2, false, FA_HD)
-        else ZLM_FA_LAUNCH(1, false, FA_HD)
+#define ZLM_FA_FORMS(X)                                                                                           \
+    if (softcap > 0.f) {                                                                                          \
+        if (hpc == 2) ZLM_FA_LAUNCH(2, true, FA_HD, X)                                                            \
+        else ZLM_FA_LAUNCH(1, true, FA_HD, X)                                                                     \
+    } else {                                                                                                      \
+        if (hpc == 2) ZLM_FA_LAUNCH(2, false, FA_HD, X)                                                           \
+        else ZLM_FA_LAUNCH(1, false, FA_HD, X)                                                                    \
     }
+    if (hd > FA_HD) {
+        if (softcap > 0.f) ZLM_FA_LAUNCH(1, true, 192, FA_PLAIN)
+        else ZLM_FA_LAUNCH(1, false, 192, FA_PLAIN)
+    } else if (bias) {
+        ZLM_FA_FORMS(FA_BIAS)
+    } else if (keep) {
+        ZLM_FA_FORMS(FA_KEEP)
+    } else {
+        ZLM_FA_FORMS(FA_PLAIN)
+    }
+#undef ZLM_FA_FORMS
 #undef ZLM_FA_LAUNCH
     return zlm_check_launch("attention_prefill_tc");
 }
@@ -554,10 +585,10 @@ extern "C" int zlm_attention_prefill_tc(void* out, int out_stride, const void* q
                                         int table_stride, const int* cu_seqlens, const int* seq_slot,
                                         const int* seq_start, int R, int max_new, int nq, int nkv, int hd,
                                         float scale, int window, int sink, int chunk, float softcap, const float* sinks,
-                                        int v_share, cudaStream_t st) {
+                                        int v_share, int keep, const float* bias, int bias_n, cudaStream_t st) {
     return zlm_attention_prefill_tc_vd(out, out_stride, q, q_stride, T, pool, pool_pages, block_table, table_stride,
                                        cu_seqlens, seq_slot, seq_start, R, max_new, nq, nkv, hd, hd, scale, window, sink,
-                                       chunk, softcap, sinks, v_share, st);
+                                       chunk, softcap, sinks, v_share, keep, bias, bias_n, st);
 }
 
 // heads of a kv group per block: 0 lets the dispatcher choose; 1 or 2 force that many where the kv

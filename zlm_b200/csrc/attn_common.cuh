@@ -40,19 +40,54 @@ __device__ __forceinline__ unsigned pack_bf16(float lo, float hi) {
 //            (null with the flag `sink` set: the number is 0)
 //   v_share  that many neighbouring key heads read one value head: a page is [nkv key heads | nkv / v_share value
 //            heads] of [ZLM_PAGE][hd] each (1: the ordinary [K | V] of nkv heads each)
+//   keep     > 0 (with a window): the sequence's first `keep` positions stay visible beside the window
+//   bias     numbers [nq][bias_n] added to the scores after scale and cap, by distance: query i reads
+//            bias[head][min(i - j, bias_n - 1)] for key j
 struct AttnOpts {
     int chunk;
     float softcap;
     const float* sinks;
     int v_share;
+    int keep;
+    const float* bias;
+    int bias_n;
 };
-static inline AttnOpts attn_no_opts() { return AttnOpts{0, 0.f, nullptr, 1}; }
+static inline AttnOpts attn_no_opts() { return AttnOpts{0, 0.f, nullptr, 1, 0, nullptr, 0}; }
+// what the entry points ask of the options they are given
+#define ZLM_REQUIRE_ATTN_OPTS(what)                                                                                   \
+    ZLM_REQUIRE(chunk >= 0 && softcap >= 0.f && v_share >= 1 && nkv % v_share == 0,                                   \
+                what ": chunk=%d softcap=%g v_share=%d", chunk, (double)softcap, v_share);                            \
+    ZLM_REQUIRE(keep >= 0 && (keep == 0 || (window > 0 && chunk == 0)), what ": %d first keys beside a window of %d", keep, window); \
+    ZLM_REQUIRE(!bias || bias_n > 0, what ": a distance bias of %d entries", bias_n)
+#define ATTN_LOG2E 1.4426950408889634f
 
 // the first key that the query at `pos` reads
 __device__ __forceinline__ int attn_first_key(int pos, int window, int chunk) {
     int lo = (window != 0 && pos + 1 > window) ? pos + 1 - window : 0;
     if (chunk > 0) lo = max(lo, pos - pos % chunk);
     return lo;
+}
+
+// The pages a tile of queries walks: the pages of the first kept keys, then those from the tile's first key on.
+//   n        how many
+//   page(w)  the w-th one's logical page; beyond the last one, pages beyond every query's position
+struct AttnWalk {
+    int kept, lo, n;
+    __device__ __forceinline__ AttnWalk(int page_lo, int page_hi, int keep) {
+        kept = keep > 0 ? min((keep + ZLM_PAGE - 1) / ZLM_PAGE, page_hi) : 0;
+        lo = keep > 0 ? max(page_lo, kept) : page_lo;
+        n = kept + page_hi - lo;
+    }
+    __device__ __forceinline__ int page(int w) const { return w < kept ? w : lo + (w - kept); }
+};
+
+// whether the query at `pos` whose window starts at `lo` reads the key
+__device__ __forceinline__ bool attn_sees(int key, int pos, int lo, int keep) { return key <= pos && (key >= lo || key < keep); }
+
+// the bias of a head (its row of the table) at a distance, in base-2 exponents
+__device__ __forceinline__ float attn_bias_log2(const float* row, int distance, int bias_n) {
+    const float* p = row + min(max(distance, 0), bias_n - 1);
+    return ZLM_CHK(p, 4) ? __ldg(p) * ATTN_LOG2E : 0.f;
 }
 
 // a raw dot product as a base-2 exponent: dot * scale * log2(e), capped first where the mixer asks for it

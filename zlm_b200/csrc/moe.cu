@@ -6,7 +6,7 @@
 //                 for a bias-free expert is the same as scaling its first product
 //   moe_down      stream[t, :] += sum_j W_down[e_tj] a[t, j, :], experts in the order they were chosen
 //   act_scale     out[t, i] = act(u[t, i]) * s[t]  (a shared expert between the library's dense products)
-// act is relu(z)^2.  A warp owns one output and shares the inner dimension among its lanes, so every sum's
+// act is relu(z)^2, or a gated form of two matrices.  A warp owns one output and shares the inner dimension among its lanes, so every sum's
 // order depends on the sizes alone, not on the batch.
 #include "common.cuh"
 
@@ -284,7 +284,7 @@ template <typename TA>
 __global__ void __launch_bounds__(MOE_WARPS * 32)
 moe_up_kernel(TA* __restrict__ act, const TA* __restrict__ x, int x_stride, const TA* __restrict__ Wup,
               const int* __restrict__ idx, const float* __restrict__ wgt, int top, int F, int K, int scale_input, int act_kind,
-              int n_real) {
+              int n_real, float limit, float alpha) {
     pdl_launch_dependents();
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int f = blockIdx.x * MOE_WARPS + warp, j = blockIdx.y, t = blockIdx.z;
@@ -301,14 +301,21 @@ moe_up_kernel(TA* __restrict__ act, const TA* __restrict__ x, int x_stride, cons
         const float z = warp_dot(Wup + ((size_t)e * F + f) * K, xr, K, lane, vec);
         a = scale_input ? relu2(w * z) : w * relu2(z);
     } else {
-        // gated: the expert's rows are [gate | up], in groups of 8 gate rows and the 8 matching up rows (act_kind 2:
-        // the layout of the products with a fused gate) or as two halves (act_kind 1)
-        const size_t rg = act_kind == 2 ? (size_t)(f / 8) * 16 + f % 8 : (size_t)f;
-        const size_t ru = act_kind == 2 ? rg + 8 : (size_t)F + f;
+        // gated: the expert's rows are [gate | up], in groups of 8 gate rows and the 8 matching up rows (act_kind 2, 4:
+        // the layout of the products with a fused gate) or as two halves (act_kind 1, 3)
+        const bool eights = (act_kind & 1) == 0;
+        const size_t rg = eights ? (size_t)(f / 8) * 16 + f % 8 : (size_t)f;
+        const size_t ru = eights ? rg + 8 : (size_t)F + f;
         float zg = warp_dot(Wup + ((size_t)e * 2 * F + rg) * K, xr, K, lane, vec);
         float zu = warp_dot(Wup + ((size_t)e * 2 * F + ru) * K, xr, K, lane, vec);
         if (scale_input) { zg *= w; zu *= w; }
-        a = zg / (1.0f + expf(-zg)) * zu;
+        if (act_kind >= 3) {                     // clamped: g sigmoid(alpha g) (u + 1)
+            zg = fminf(zg, limit);
+            zu = fminf(fmaxf(zu, -limit), limit);
+            a = zg / (1.0f + expf(-alpha * zg)) * (zu + 1.0f);
+        } else {
+            a = zg / (1.0f + expf(-zg)) * zu;
+        }
         if (!scale_input) a *= w;
     }
     if (lane == 0 && ZLM_CHK(act + ((size_t)t * top + j) * F + f, sizeof(TA)))
@@ -344,20 +351,22 @@ moe_down_kernel(float* __restrict__ stream, const TA* __restrict__ act, const TA
 }
 
 // act_kind 0: relu(z)^2 of one matrix [E][F][K]; 1: silu(gate) * up of [E][2F][K], gate rows then up rows; 2: the same
-// with the rows in groups of 8 gate and 8 up.  n_real: experts from this index on are identity experts (no matrices).
+// with the rows in groups of 8 gate and 8 up; 3 and 4: the same two layouts with g sigmoid(alpha g) (u + 1), g =
+// min(gate, limit), u = clamp(up, -limit, limit).  n_real: experts from this index on are identity experts (no matrices).
 extern "C" int zlm_moe_up(void* act, const void* x, int x_stride, const void* Wup, const int* idx, const float* wgt,
-                          int dtype, int T, int top, int F, int K, int scale_input, int act_kind, int n_real,
-                          cudaStream_t st) {
+                          int dtype, int T, int top, int F, int K, int scale_input, int act_kind, int n_real, float limit,
+                          float alpha, cudaStream_t st) {
     if (T == 0) return ZLM_OK;
-    ZLM_REQUIRE(act_kind >= 0 && act_kind <= 2 && (act_kind != 2 || F % 8 == 0), "moe_up: activation %d with F=%d", act_kind, F);
+    ZLM_REQUIRE(act_kind >= 0 && act_kind <= 4 && ((act_kind != 2 && act_kind != 4) || F % 8 == 0) && (act_kind < 3 || limit > 0.f),
+                "moe_up: activation %d with F=%d, limit %g", act_kind, F, (double)limit);
     ZLM_REQUIRE(T <= 65535 && top > 0 && top <= 65535 && F > 0 && K > 0, "moe_up: bad sizes T=%d top=%d F=%d K=%d", T, top, F, K);
     dim3 grid((F + MOE_WARPS - 1) / MOE_WARPS, top, T);
     if (dtype == ZLM_DTYPE_F32)
         zlm_launch(moe_up_kernel<float>, grid, MOE_WARPS * 32, 0, st, (float*)act, (const float*)x, x_stride,
-                   (const float*)Wup, idx, wgt, top, F, K, scale_input, act_kind, n_real);
+                   (const float*)Wup, idx, wgt, top, F, K, scale_input, act_kind, n_real, limit, alpha);
     else if (dtype == ZLM_DTYPE_BF16)
         zlm_launch(moe_up_kernel<__nv_bfloat16>, grid, MOE_WARPS * 32, 0, st, (__nv_bfloat16*)act, (const __nv_bfloat16*)x,
-                   x_stride, (const __nv_bfloat16*)Wup, idx, wgt, top, F, K, scale_input, act_kind, n_real);
+                   x_stride, (const __nv_bfloat16*)Wup, idx, wgt, top, F, K, scale_input, act_kind, n_real, limit, alpha);
     else
         ZLM_REQUIRE(false, "moe_up: unsupported dtype %d", dtype);
     return zlm_check_launch("moe_up");

@@ -287,13 +287,24 @@ extern "C" int zlm_head_gate(void* out, int out_stride, const void* o, int o_is_
 //   a short causal convolution per channel (as above; has_conv 0: none),
 //   a norm of q and k: per head without weight (norm_mode 1), per head with one weight of `dim` shared by the heads
 //   (2), or over the whole projection at once, all heads of q (of k) together, with a weight per channel (3),
-//   rotation of the first n_rot coordinates of every q and k head, coordinate i against i + n_rot/2, by the angle
-//   pos * inv_freq[i]; cosine and sine are multiplied by rot_scale (a frequency table scaled for long contexts
-//   carries such a factor),
+//   rotation of the first n_rot coordinates of every q and k head, coordinate i against i + n_rot/2 (or, interleaved,
+//   2i against 2i + 1), by the angle pos * inv_freq[i]; cosine and sine are multiplied by rot_scale (a frequency table
+//   scaled for long contexts carries such a factor),
+//   a temperature on q: times 1 + coef * ln(floor((pos + 1) / every) + 1),
+//   a mixture of values between layers: v <- (1 - lambda) v + lambda v_first, v_first [T][nkv*vdim] the values that an
+//   earlier layer's preparation of the same step left (a layer leaves its own, unmixed, where it is given v_keep),
 //   q written head by head, k and v into the token's place of the paged cache, heads padded with zeros to hdp.
 // A block per token: the token's convolved channels are held in shared memory as fp32, the sums of squares are
 // block sums in a fixed order, angles, cosines and sines are fp32.
 #define AP_THREADS 256
+struct AttnPrepExtras {
+    int interleaved;          // rotation of neighbouring coordinates
+    float temp_coef;          // 0: no temperature
+    int temp_every;
+    const void* v_first;      // null: values as they are
+    float lambda;
+    void* v_keep;             // null: nobody mixes this layer's values in
+};
 template <typename TA>
 __global__ void __launch_bounds__(AP_THREADS)
 attn_prep_kernel(TA* __restrict__ q_out, int q_out_stride, const TA* __restrict__ proj, int proj_stride,
@@ -301,7 +312,7 @@ attn_prep_kernel(TA* __restrict__ q_out, int q_out_stride, const TA* __restrict_
                  const int* __restrict__ token_slot, const int* __restrict__ token_seq, const int* __restrict__ seq_start,
                  const int* __restrict__ cu_seqlens, const int* __restrict__ block_table, int table_stride,
                  TA* __restrict__ pool, int nq, int nkv, int dim, int vdim, int hdp, int taps, int norm_mode, VecW q_w,
-                 VecW k_w, float eps, const float* __restrict__ inv_freq, int n_rot, float rot_scale) {
+                 VecW k_w, float eps, const float* __restrict__ inv_freq, int n_rot, float rot_scale, AttnPrepExtras ex) {
     extern __shared__ float ap_smem[];          // [C] channels, [nq + nkv] inverse root mean squares, [32] reduction
     pdl_trigger();
     const int t = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
@@ -365,6 +376,7 @@ attn_prep_kernel(TA* __restrict__ q_out, int q_out_stride, const TA* __restrict_
     int page = 0;
     if (ZLM_CHK(block_table + (size_t)slot * table_stride + pos / ZLM_PAGE, 4))
         page = block_table[(size_t)slot * table_stride + pos / ZLM_PAGE];
+    const float temp = ex.temp_coef != 0.f ? fmaf(ex.temp_coef, logf((float)((pos + 1) / ex.temp_every) + 1.0f), 1.0f) : 1.0f;
     // (steps of few tokens run several blocks a token: each repeats the sums above and writes its share)
     for (int x = blockIdx.y * AP_THREADS + tid; x < (nq + 2 * nkv) * hdp; x += AP_THREADS * gridDim.y) {
         const int unit = x / hdp, e = x - unit * hdp;
@@ -377,15 +389,26 @@ attn_prep_kernel(TA* __restrict__ q_out, int q_out_stride, const TA* __restrict_
                 const float sc = inv[unit];
                 o = val[c] * sc * (norm_mode >= 2 ? w[wb + e] : 1.0f);
                 if (e < n_rot) {
-                    const int fi = e < half ? e : e - half;
-                    const int pe = e < half ? e + half : e - half;
+                    const bool first = ex.interleaved ? (e & 1) == 0 : e < half;
+                    const int fi = ex.interleaved ? e >> 1 : (first ? e : e - half);
+                    const int pe = ex.interleaved ? e ^ 1 : (first ? e + half : e - half);
                     const float other = val[unit * dim + pe] * sc * (norm_mode >= 2 ? w[wb + pe] : 1.0f);
                     const float cs = rot[fi], sn = rot[half + fi];
-                    o = e < half ? o * cs - other * sn : o * cs + other * sn;
+                    o = first ? o * cs - other * sn : o * cs + other * sn;
                 }
+                if (unit < nq) o *= temp;
             }
         } else if (e < vdim) {
-            o = val[QC + KC + (unit - nq - nkv) * vdim + e];
+            const int c = (unit - nq - nkv) * vdim + e;
+            o = val[QC + KC + c];
+            if (ex.v_keep) {
+                TA* keep = (TA*)ex.v_keep + (size_t)t * nkv * vdim + c;
+                if (ZLM_CHK(keep, sizeof(TA))) *keep = from_f32<TA>(o);
+            }
+            if (ex.v_first) {
+                const TA* vf = (const TA*)ex.v_first + (size_t)t * nkv * vdim + c;
+                if (ZLM_CHK(vf, sizeof(TA))) o = (1.0f - ex.lambda) * o + ex.lambda * to_f32(*vf);
+            }
         }
         TA* dst;
         if (unit < nq) {
@@ -404,7 +427,8 @@ static void launch_attn_prep(void* q_out, int q_out_stride, const void* proj, in
                              const int* token_pos, const int* token_slot, const int* token_seq, const int* seq_start,
                              const int* cu_seqlens, const int* seq_slot, const int* block_table, int table_stride, void* pool,
                              int T, int R, int nq, int nkv, int dim, int vdim, int hdp, int taps, int norm_mode, VecW q_w,
-                             VecW k_w, float eps, const float* inv_freq, int n_rot, float rot_scale, cudaStream_t st) {
+                             VecW k_w, float eps, const float* inv_freq, int n_rot, float rot_scale, AttnPrepExtras ex,
+                             cudaStream_t st) {
     const int C = (nq + nkv) * dim + nkv * vdim;
     const size_t smem = (size_t)(C + nq + nkv + 32 + n_rot) * sizeof(float);
     // blocks a token: one where the tokens alone fill the device, else as many as give it two rounds of work
@@ -414,7 +438,7 @@ static void launch_attn_prep(void* q_out, int q_out_stride, const void* proj, in
     zlm_launch(attn_prep_kernel<TA>, dim3(T, share), dim3(AP_THREADS), smem, st, (TA*)q_out, q_out_stride, (const TA*)proj,
                proj_stride, (const TA*)conv_w, (const TA*)state, token_pos, token_slot, token_seq, seq_start, cu_seqlens,
                block_table, table_stride, (TA*)pool, nq, nkv, dim, vdim, hdp, taps, norm_mode, q_w, k_w, eps, inv_freq, n_rot,
-               rot_scale);
+               rot_scale, ex);
     if (conv_w && taps > 1)
         zlm_launch(conv_state_update_kernel<TA>, dim3(R, (C + 255) / 256), dim3(256), 0, st, (TA*)state, (const TA*)proj,
                    proj_stride, seq_slot, cu_seqlens, C, taps);
@@ -422,14 +446,19 @@ static void launch_attn_prep(void* q_out, int q_out_stride, const void* proj, in
 
 // As zlm_conv_norm_write, with: conv_w null for no convolution; norm_mode 0 none, 1 per head without weight, 2 per
 // head with q_w / k_w [dim], 3 over all heads at once with q_w [nq*dim] / k_w [nkv*dim]; inv_freq [n_rot/2] fp32
-// (n_rot 0: no rotation); rot_scale multiplies cosines and sines.
+// (n_rot 0: no rotation; interleaved: neighbouring coordinates are a pair); rot_scale multiplies cosines and sines;
+// temp_coef, temp_every: the temperature on q (coef 0: none); v_first, lambda: the values mixed in (null: none); v_keep:
+// where this layer leaves its own values (null: nowhere).
 extern "C" int zlm_attn_prep(void* q_out, int q_out_stride, const void* proj, int proj_stride, const void* conv_w,
                              void* state, int dtype, const int* token_pos, const int* token_slot, const int* token_seq,
                              const int* seq_start, const int* cu_seqlens, const int* seq_slot, const int* block_table,
                              int table_stride, void* pool, int T, int R, int nq, int nkv, int dim, int vdim, int hdp,
                              int taps, int norm_mode, const void* q_w, const void* k_w, int w_dtype, float eps,
-                             const float* inv_freq, int n_rot, float rot_scale, cudaStream_t st) {
+                             const float* inv_freq, int n_rot, float rot_scale, int interleaved, float temp_coef, int temp_every,
+                             const void* v_first, float lambda, void* v_keep, cudaStream_t st) {
     if (T == 0) return ZLM_OK;
+    ZLM_REQUIRE(temp_coef == 0.f || temp_every > 0, "attn_prep: a temperature that changes every %d positions", temp_every);
+    const AttnPrepExtras ex{interleaved, temp_coef, temp_every, v_first, lambda, v_keep};
     ZLM_REQUIRE(nq > 0 && nkv > 0 && dim > 0 && vdim > 0 && hdp >= dim && hdp >= vdim, "attn_prep: heads %d/%d of %d and %d columns padded to %d",
                 nq, nkv, dim, vdim, hdp);
     ZLM_REQUIRE(taps >= 1 && taps <= SC_MAX_TAPS, "attn_prep: %d taps (at most %d)", taps, SC_MAX_TAPS);
@@ -447,7 +476,7 @@ extern "C" int zlm_attn_prep(void* q_out, int q_out_stride, const void* proj, in
         }
         launch_attn_prep<float>(q_out, q_out_stride, proj, proj_stride, conv_w, state, token_pos, token_slot, token_seq, seq_start,
                                 cu_seqlens, seq_slot, block_table, table_stride, pool, T, R, nq, nkv, dim, vdim, hdp, taps,
-                                norm_mode, qw, kw, eps, inv_freq, n_rot, rot_scale, st);
+                                norm_mode, qw, kw, eps, inv_freq, n_rot, rot_scale, ex, st);
     } else if (dtype == ZLM_DTYPE_BF16) {
         static bool big[64] = {};
         if (smem > 48 * 1024 && !big[zlm_device_index()]) {
@@ -456,7 +485,7 @@ extern "C" int zlm_attn_prep(void* q_out, int q_out_stride, const void* proj, in
         }
         launch_attn_prep<__nv_bfloat16>(q_out, q_out_stride, proj, proj_stride, conv_w, state, token_pos, token_slot, token_seq,
                                         seq_start, cu_seqlens, seq_slot, block_table, table_stride, pool, T, R, nq, nkv, dim,
-                                        vdim, hdp, taps, norm_mode, qw, kw, eps, inv_freq, n_rot, rot_scale, st);
+                                        vdim, hdp, taps, norm_mode, qw, kw, eps, inv_freq, n_rot, rot_scale, ex, st);
     } else {
         ZLM_REQUIRE(false, "attn_prep: unsupported dtype %d", dtype);
     }

@@ -701,7 +701,8 @@ class CudaKernels:
                   token_pos: torch.Tensor, token_slot: torch.Tensor, nq: int, nkv: int, hd: int,
                   scale: float, window: int, plan=None, len_bucket: Optional[int] = None,
                   v_dim: Optional[int] = None, sink: bool = False, chunk: int = 0, softcap: float = 0.0,
-                  sinks: Optional[torch.Tensor] = None, v_share: int = 1) -> None:
+                  sinks: Optional[torch.Tensor] = None, v_share: int = 1, keep: int = 0,
+                  bias: Optional[torch.Tensor] = None) -> None:
         """out[t, h] = softmax(q[t, h] . K * scale) V over the keys [start, pos[t]] of the
         token's slot; q may be a column view of the fused qkv buffer.  ``plan`` is the
         step's context (one token per sequence: the split-KV kernel; whole prompts or
@@ -712,8 +713,15 @@ class CudaKernels:
         only the keys of its own chunk of that many positions (counted from position 0 of the sequence).
         ``softcap``: scores become softcap * tanh(score / softcap) after the scale.  ``v_share``: that many
         neighbouring key heads read one value head; a page of the pool is then [nkv key heads | nkv / v_share
-        value heads] of [PAGE_TOKENS, hd] each (with 1, the ordinary [2, nkv, PAGE_TOKENS, hd])."""
+        value heads] of [PAGE_TOKENS, hd] each (with 1, the ordinary [2, nkv, PAGE_TOKENS, hd]).  ``keep``: with a
+        window, the sequence's first ``keep`` keys stay visible beside it.  ``bias`` [nq, n] fp32: added to the scores
+        after scale and cap, bias[h, min(distance, n - 1)]."""
         T = q.shape[0]
+        bias_n = 0
+        if bias is not None:
+            assert bias.dtype == torch.float32 and bias.dim() == 2 and bias.shape[0] == nq and bias.is_contiguous()
+            bias_n = int(bias.shape[1])
+        assert keep >= 0 and (keep == 0 or (window > 0 and not chunk))
         if sinks is not None:
             assert sinks.dtype == torch.float32 and sinks.shape == (nq,) and sinks.is_contiguous()
             sink = True
@@ -722,7 +730,7 @@ class CudaKernels:
         assert q.stride(1) == 1 and out.stride(1) == 1 and pool.is_contiguous()
         assert v_share >= 1 and nkv % v_share == 0 and chunk >= 0 and softcap >= 0
         assert pool[0].numel() == (nkv + nkv // v_share) * PAGE_TOKENS * hd and pool.shape[-1] == hd
-        extra = (c_int(chunk), c_float(softcap), self._p(sinks), c_int(v_share))
+        extra = (c_int(chunk), c_float(softcap), self._p(sinks), c_int(v_share), c_int(keep), self._p(bias), c_int(bias_n))
         if (plan is not None and plan.is_decode and q.dtype == torch.bfloat16
                 and self.lib.zlm_attention_decode_supported(nq, nkv, hd)):
             if len_bucket is None:
@@ -746,7 +754,8 @@ class CudaKernels:
                 and getattr(plan, "cu_seqlens", None) is not None
                 and self.lib.zlm_attention_prefill_supported(nq, nkv, hd)):
             impl = getattr(plan, "attention_impl", None)
-            if impl != "mma" and self.lib.zlm_attention_prefill_tc_supported(nq, nkv, hd, q.stride(0), out.stride(0)):
+            if (impl != "mma" and not (keep and bias is not None)
+                    and self.lib.zlm_attention_prefill_tc_supported(nq, nkv, hd, q.stride(0), out.stride(0))):
                 self._call("zlm_attention_prefill_tc", self._p(out), c_int(out.stride(0)),
                            self._p(q), c_int(q.stride(0)), c_int(T), self._p(pool),
                            ctypes.c_longlong(pool.shape[0]), self._p(block_table),
@@ -755,7 +764,7 @@ class CudaKernels:
                            c_int(plan.max_new), c_int(nq), c_int(nkv), c_int(hd), c_float(scale), c_int(window),
                            sk, *extra, self._stream())
                 return
-            if (impl != "mma" and v_dim is not None and v_dim < hd
+            if (impl != "mma" and v_dim is not None and v_dim < hd and not keep and bias is None
                     and self.lib.zlm_attention_prefill_tc_vd_supported(nq, nkv, hd, v_dim, q.stride(0), out.stride(0))):
                 # keys of 192 over values of 128 on the tcgen05 kernel (out's columns from v_dim on become zeros)
                 self._call("zlm_attention_prefill_tc_vd", self._p(out), c_int(out.stride(0)),
@@ -869,15 +878,22 @@ class CudaKernels:
     def attn_prep(self, q_out: torch.Tensor, proj: torch.Tensor, conv_w: Optional[torch.Tensor], state: Optional[torch.Tensor],
                   plan, block_table: torch.Tensor, pool: torch.Tensor, nq: int, nkv: int, dim: int, vdim: int, taps: int,
                   norm: str, q_w: Optional[torch.Tensor], k_w: Optional[torch.Tensor], eps: float,
-                  inv_freq: Optional[torch.Tensor], n_rot: int, rot_scale: float = 1.0) -> None:
+                  inv_freq: Optional[torch.Tensor], n_rot: int, rot_scale: float = 1.0, interleaved: bool = False,
+                  q_temp: Optional[tuple] = None, v_first: Optional[torch.Tensor] = None, v_lambda: float = 0.0,
+                  v_keep: Optional[torch.Tensor] = None) -> None:
         """``conv_norm_write`` in its general form: the convolution is optional (``conv_w`` None), the norm of q and k is
         "none", "unit" (per head, no weight), "head" (per head, weights ``q_w`` / ``k_w`` [dim] shared by the heads) or
         "row" (over all heads of q, and of k, at once, weights [nq*dim] / [nkv*dim]), and the first ``n_rot`` coordinates
         of every q and k head are rotated (i against i + n_rot/2) by pos * inv_freq[i], cosines and sines times
-        ``rot_scale``."""
+        ``rot_scale`` (``interleaved``: 2i against 2i + 1).  ``q_temp`` (coef, every): q is multiplied by
+        1 + coef * ln(floor((pos + 1) / every) + 1).  ``v_first`` [T, nkv*vdim]: v becomes (1 - v_lambda) v + v_lambda
+        v_first.  ``v_keep`` [T, nkv*vdim] receives v as it was before that."""
         T = proj.shape[0]
         hdp = pool.shape[-1]
         C = (nq + nkv) * dim + nkv * vdim
+        for v in (v_first, v_keep):
+            assert v is None or (v.shape == (T, nkv * vdim) and v.dtype == proj.dtype and v.is_contiguous())
+        coef, every = q_temp if q_temp is not None else (0.0, 1)
         mode = {"none": 0, "unit": 1, "head": 2, "row": 3}[norm]
         assert proj.shape[1] >= C and proj.stride(1) == 1 and q_out.shape == (T, nq * hdp) and q_out.stride(1) == 1
         assert tuple(pool.shape[1:]) == (2, nkv, PAGE_TOKENS, hdp) and pool.is_contiguous() and block_table.dtype == torch.int32
@@ -903,7 +919,8 @@ class CudaKernels:
                    self._p(pool), c_int(T), c_int(plan.R), c_int(nq), c_int(nkv), c_int(dim), c_int(vdim), c_int(hdp),
                    c_int(taps), c_int(mode), self._p(q_w if mode >= 2 else None), self._p(k_w if mode >= 2 else None),
                    c_int(_dt(q_w) if mode >= 2 else F32), c_float(eps), self._p(inv_freq if n_rot else None), c_int(n_rot),
-                   c_float(rot_scale), self._stream())
+                   c_float(rot_scale), c_int(1 if interleaved else 0), c_float(coef), c_int(every), self._p(v_first),
+                   c_float(v_lambda), self._p(v_keep), self._stream())
 
     def norm_gate(self, out: torch.Tensor, o: torch.Tensor, g: Optional[torch.Tensor], heads: int, v_dim: int, group: str,
                   weight: Optional[torch.Tensor], eps: float, act: str, out_scale: float = 1.0) -> None:
@@ -1015,6 +1032,55 @@ class CudaKernels:
                    c_int(x_off), c_int(g_off), self._p(bz), self._p(bx), c_int(_dt(b) if b is not None else F32), self._p(state),
                    c_int(_dt(proj)), self._p(plan.seq_slot), self._p(plan.cu_seqlens), c_int(T), c_int(plan.R), c_int(W),
                    c_int(1 if cluster else 0), self._stream())
+
+    def mlstm_step(self, out: torch.Tensor, proj: torch.Tensor, q_off: int, k_off: int, v_off: int, g_off: int, z: torch.Tensor,
+                   i_off: int, f_off: int, b_i: Optional[torch.Tensor], b_f: Optional[torch.Tensor], cap: float,
+                   state, plan, heads: int, dim: int, v_dim: int, q_scale: float, w_norm: torch.Tensor, eps: float) -> None:
+        """One token of a matrix memory (see ``mlstm``) for every sequence of a decode step, with what follows it:
+        out [T, heads*v_dim] = o / rms(o, per head) * w_norm * sigmoid(g), g the columns of ``proj`` from g_off on."""
+        T, N = out.shape
+        S, n, m = self._check_mlstm(proj, z, b_i, b_f, state, heads, dim, v_dim)
+        assert plan.is_decode and plan.R == T and N == heads * v_dim and out.stride(1) == 1
+        assert w_norm.shape == (N,) and w_norm.is_contiguous()
+        b = b_i if b_i is not None else b_f
+        self._call("zlm_mlstm_step", self._p(out), c_int(out.stride(0)), c_int(_dt(out)), self._p(proj), c_int(proj.stride(0)),
+                   c_int(_dt(proj)), c_int(q_off), c_int(k_off), c_int(v_off), c_int(g_off), self._p(z), c_int(z.stride(0)),
+                   c_int(i_off), c_int(f_off), self._p(b_i), self._p(b_f), c_int(_dt(b) if b is not None else F32), c_float(cap),
+                   self._p(S), self._p(n), self._p(m), self._p(plan.seq_slot), self._p(plan.cu_seqlens), c_int(plan.R),
+                   c_int(heads), c_int(dim), c_int(v_dim), c_float(q_scale), self._p(w_norm), c_int(_dt(w_norm)), c_float(eps),
+                   self._stream())
+
+    def mlstm(self, o: torch.Tensor, proj: torch.Tensor, q_off: int, k_off: int, v_off: int, z: torch.Tensor, i_off: int,
+              f_off: int, b_i: Optional[torch.Tensor], b_f: Optional[torch.Tensor], cap: float, state, plan, heads: int,
+              dim: int, v_dim: int, q_scale: float) -> None:
+        """o [T, heads*v_dim] fp32: per head, with i = cap tanh((zi + b_i) / cap), f = log sigmoid(cap tanh((zf + b_f) / cap)),
+        m_t = max(f + m_(t-1), i), S_t = exp(f + m_(t-1) - m_t) S_(t-1) + exp(i - m_t) k v^T and n_t likewise with k alone,
+        o = S_t^T q / (max(|n_t . q|, exp(-m_t)) + 1e-6).  q (times ``q_scale``), k, v are columns of ``proj`` from q_off,
+        k_off, v_off on; zi and zf columns i_off + h and f_off + h of ``z`` (fp32); ``state`` (S [slots, heads, dim, v_dim],
+        n [slots, heads, dim], m [slots, heads]), all fp32.  A sequence's tokens run in pieces side by side."""
+        T = proj.shape[0]
+        S, n, m = self._check_mlstm(proj, z, b_i, b_f, state, heads, dim, v_dim)
+        assert o.shape == (T, heads * v_dim) and o.dtype == torch.float32 and o.is_contiguous()
+        max_new = int(plan.max_new)
+        self.lib.zlm_mlstm_scratch.restype = ctypes.c_longlong
+        part = plan.scratch("mlstm.pieces", (int(self.lib.zlm_mlstm_scratch(plan.R, heads, dim, v_dim, max_new)),), torch.float32)
+        b = b_i if b_i is not None else b_f
+        self._call("zlm_mlstm", self._p(o), self._p(proj), c_int(proj.stride(0)), c_int(_dt(proj)), c_int(q_off), c_int(k_off),
+                   c_int(v_off), self._p(z), c_int(z.stride(0)), c_int(i_off), c_int(f_off), self._p(b_i), self._p(b_f),
+                   c_int(_dt(b) if b is not None else F32), c_float(cap), self._p(S), self._p(n), self._p(m),
+                   self._p(plan.seq_slot), self._p(plan.cu_seqlens), c_int(T), c_int(plan.R), c_int(heads), c_int(dim),
+                   c_int(v_dim), c_float(q_scale), c_int(max_new), self._p(part), self._stream())
+
+    @staticmethod
+    def _check_mlstm(proj, z, b_i, b_f, state, heads, dim, v_dim):
+        S, n, m = state
+        assert proj.stride(1) == 1 and z.dtype == torch.float32 and z.stride(1) == 1 and z.shape[0] == proj.shape[0]
+        assert tuple(S.shape[1:]) == (heads, dim, v_dim) and tuple(n.shape[1:]) == (heads, dim) and tuple(m.shape[1:]) == (heads,)
+        for t in (S, n, m):
+            assert t.dtype == torch.float32 and t.is_contiguous()
+        for b in (b_i, b_f):
+            assert b is None or (b.shape == (heads,) and b.is_contiguous() and b.dtype == (b_i if b_i is not None else b_f).dtype)
+        return S, n, m
 
     def lowrank_decay(self, alpha: torch.Tensor, proj: torch.Tensor, lo_off: int, w2: torch.Tensor, b: Optional[torch.Tensor],
                       tau: float) -> None:
@@ -1478,13 +1544,15 @@ class CudaKernels:
                    c_int({"sigmoid": 0, "softmax": 1}[score]), c_int(1 if renormalize else 0),
                    *self._route_extras(correction, experts, groups, keep, weight_scale, group_top), self._stream())
 
-    _ACT_KINDS = {"relu2": 0, "swiglu": 1, "swiglu_interleaved": 2}
+    _ACT_KINDS = {"relu2": 0, "swiglu": 1, "swiglu_interleaved": 2, "swish_limit": 3, "swish_limit_interleaved": 4}
 
     def moe_up(self, act: torch.Tensor, x: torch.Tensor, w_up: torch.Tensor, idx: torch.Tensor, wgt: torch.Tensor,
-               scale_input: bool = True, activation: str = "relu2") -> None:
+               scale_input: bool = True, activation: str = "relu2", limit: float = 0.0, alpha: float = 1.702) -> None:
         """act[t, j, :] = relu(W_up[idx[t, j]] (wgt[t, j] x[t]))^2 (``scale_input``), or wgt[t, j] * relu(W_up[..] x[t])^2;
         w_up [experts, F, K], act [T, top, F].  ``activation`` "swiglu": w_up is [experts, 2F, K], an expert's gate rows then
-        its up rows, and the activation is silu(gate) * up ("swiglu_interleaved": the rows in groups of 8 gate, 8 up).
+        its up rows, and the activation is silu(gate) * up ("swiglu_interleaved": the rows in groups of 8 gate, 8 up);
+        "swish_limit" and "swish_limit_interleaved": the same layouts with g sigmoid(alpha g) (u + 1), g = min(gate, limit),
+        u = clamp(up, -limit, limit).
         A choice of an index from ``experts`` on (an identity expert) writes nothing."""
         T, K = x.shape
         top = idx.shape[1]
@@ -1495,7 +1563,7 @@ class CudaKernels:
         assert x.dtype == w_up.dtype == act.dtype and x.stride(1) == 1
         self._call("zlm_moe_up", self._p(act), self._p(x), c_int(x.stride(0)), self._p(w_up), self._p(idx), self._p(wgt),
                    c_int(_dt(x)), c_int(T), c_int(top), c_int(F), c_int(K), c_int(1 if scale_input else 0), c_int(kind),
-                   c_int(E), self._stream())
+                   c_int(E), c_float(limit), c_float(alpha), self._stream())
 
     def moe_down(self, stream: torch.Tensor, act: torch.Tensor, w_down: torch.Tensor, idx: torch.Tensor,
                  identity_input: Optional[torch.Tensor] = None, wgt: Optional[torch.Tensor] = None) -> None:
@@ -1514,20 +1582,21 @@ class CudaKernels:
 
     def moe_grouped(self, stream: torch.Tensor, x: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tensor,
                     idx: torch.Tensor, wgt: torch.Tensor, scale_input: bool = True, impl: Optional[str] = None,
-                    activation: str = "relu2", identity: bool = False) -> None:
+                    activation: str = "relu2", identity: bool = False, limit: float = 0.0, alpha: float = 1.702) -> None:
         """What ``moe_up`` and ``moe_down`` compute, for steps of many tokens (bf16): the (token, choice) pairs
         are sorted by expert on the device and every expert's rows go through its matrices as tiles of one
         grouped tensor-core product, so an expert's weights are read once per tile, not once per token.  Two
         forms (``impl`` forces one): "tc", TMA + tcgen05 on tiles of 128 rows, where an expert gets about half
         a tile or more; "mma", mma.sync on tiles of 16 to 128 rows, for fewer rows an expert.  ``activation``
         "swiglu_interleaved": w_up is [E, 2F, K], an expert's rows in sixteens of 8 gate and 8 up rows, and the first
-        product's epilogue writes silu(gate) * up ("tc" only).  ``identity``: a choice of an index from E on adds
+        product's epilogue writes silu(gate) * up ("tc" only); "swish_limit_interleaved": the same layout with ``moe_up``'s
+        clamped activation.  ``identity``: a choice of an index from E on adds
         wgt * x[t] and takes no row of any product."""
         T, K = x.shape
         E, _, F = w_down.shape
         top = idx.shape[1]
-        gated = activation == "swiglu_interleaved"
-        assert activation in ("relu2", "swiglu_interleaved")
+        gated = activation != "relu2"
+        assert activation in ("relu2", "swiglu_interleaved", "swish_limit_interleaved")
         assert x.dtype == w_up.dtype == w_down.dtype == torch.bfloat16 and x.stride(1) == 1
         assert w_up.shape == (E, F * (2 if gated else 1), K) and w_down.shape == (E, K, F) and w_up.is_contiguous() and w_down.is_contiguous()
         assert stream.dtype == torch.float32 and stream.shape == (T, K) and stream.is_contiguous()
@@ -1552,8 +1621,12 @@ class CudaKernels:
             self._call("zlm_moe_sort_padded", self._p(idx), c_int(P), c_int(E), c_int(tiles), self._p(ints), self._stream())
             self._call("zlm_moe_gather", self._p(xs), self._p(x), c_int(x.stride(0)), self._p(perm), self._p(wgt), c_int(rows),
                        c_int(top), c_int(K), c_int(1 if scale_input else 0), self._stream())
+            if activation == "swish_limit_interleaved":
+                assert limit > 0
+                self._call("zlm_set_gate_gemm_tcgen05", c_float(limit), c_float(alpha), self._stream())
             self._call("zlm_gemm_tc_grouped", self._p(act), self._p(xs), self._p(w_up), self._p(table), c_int(tiles), c_int(E),
-                       c_int(2 * F if gated else F), c_int(K), c_int(F), c_int(3 if gated else 6), self._stream())
+                       c_int(2 * F if gated else F), c_int(K), c_int(F),
+                       c_int({"relu2": 6, "swiglu_interleaved": 3, "swish_limit_interleaved": GATED_LIMIT}[activation]), self._stream())
             self._call("zlm_gemm_tc_grouped", self._p(y), self._p(act), self._p(w_down), self._p(table), c_int(tiles), c_int(E),
                        c_int(K), c_int(F), c_int(K), c_int(2), self._stream())
             self._call("zlm_moe_combine", self._p(stream), self._p(y), self._p(inv), self._p(None if scale_input else wgt),

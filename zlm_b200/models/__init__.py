@@ -5,3 +5,4 @@ from . import zekazen   # noqa: F401
 from . import lodevik   # noqa: F401
 from . import sudupel   # noqa: F401
 from . import murilix   # noqa: F401
+from . import lolivik   # noqa: F401

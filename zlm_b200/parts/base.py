@@ -68,7 +68,8 @@ class CacheRequest:
     ``chunk``: queries read only the keys of their own chunk of that many positions (counted from position 0), so the
     pages of the chunks before may be given back like those that left a window.  ``value_heads``: keys and values have
     different numbers of heads (several key heads read one value head); a page is then
-    [num_kv_heads key heads | value_heads value heads] of [PAGE_TOKENS, head_dim] each."""
+    [num_kv_heads key heads | value_heads value heads] of [PAGE_TOKENS, head_dim] each.  ``keep``: beside the window
+    queries read the first ``keep`` keys of the sequence, whose pages therefore stay."""
     num_kv_heads: int
     head_dim: int
     window: int = 0
@@ -76,6 +77,7 @@ class CacheRequest:
     dtype: Optional[torch.dtype] = None
     chunk: int = 0
     value_heads: Optional[int] = None
+    keep: int = 0
 
 
 @dataclass(frozen=True)

@@ -12,6 +12,11 @@ shared expert that every token uses.
 
 Options that other designs use:
     ``activation="swiglu"``    expert(u) = W_down (silu(W_gate u) * W_up u)     (tensors ``e<i>.gate``, ``e<i>.up``, ``e<i>.down``)
+    ``activation="swish_limit"`` the same matrices with g sigmoid(alpha g) (v + 1), g = min(W_gate u, limit), v = clamp(W_up u,
+                               -limit, limit)
+    ``shared``                 with gated experts: the shared expert is the gated feed-forward of these parameters
+                               (``swiglu``'s, ``intermediate_size`` among them; tensors ``shared.gate``, ``shared.up``,
+                               ``shared.down``) and is added as it is
     ``correction``             a vector (tensor ``correction``) added to the scores for the choice only; the weights
                                are the scores without it
     ``groups``, ``keep``       the experts form ``groups`` equal groups of neighbours; a group's mark is its largest
@@ -27,12 +32,13 @@ kernel reaches an expert by its index; the checkpoint has them one by one (``e<i
 """
 from __future__ import annotations
 
-from typing import Dict
+from typing import Any, Dict, Mapping, Optional
 
 import torch
 
 from ..registry import register_feed_forward
 from .base import FeedForward, ParamSpec, StepContext
+from .mlp import SwiGLU
 
 
 @register_feed_forward("none")
@@ -52,7 +58,8 @@ class RoutedExperts(FeedForward):
     def __init__(self, hidden_size: int, num_experts: int, top_k: int, expert_ff: int, shared_ff: int = 0,
                  shared_gate: bool = True, score: str = "sigmoid", renormalize: bool = False,
                  weight_on: str = "input", activation: str = "relu2", correction: bool = False, groups: int = 1,
-                 keep: int = 1, route_scale: float = 1.0, identity: int = 0, group_mark: str = "max"):
+                 keep: int = 1, route_scale: float = 1.0, identity: int = 0, group_mark: str = "max", limit: float = 0.0,
+                 alpha: float = 1.702, shared: Optional[Mapping[str, Any]] = None):
         self.hidden, self.E, self.top, self.F = int(hidden_size), int(num_experts), int(top_k), int(expert_ff)
         self.SF, self.shared_gate = int(shared_ff), bool(shared_gate) and int(shared_ff) > 0
         if not 0 < self.top <= self.E + int(identity):
@@ -60,9 +67,15 @@ class RoutedExperts(FeedForward):
         if score not in ("sigmoid", "softmax") or weight_on not in ("input", "output"):
             raise ValueError(f"routed experts: score={score!r}, weight_on={weight_on!r}")
         self.score, self.renormalize, self.scale_input = score, bool(renormalize), weight_on == "input"
-        if activation not in ("relu2", "swiglu"):
+        if activation not in ("relu2", "swiglu", "swish_limit"):
             raise ValueError(f"routed experts: activation={activation!r}")
-        self.activation, self.has_correction = activation, bool(correction)
+        self.limit, self.alpha = float(limit), float(alpha)
+        if activation == "swish_limit" and not self.limit > 0:
+            raise ValueError(f"routed experts: limit={limit!r}")
+        if (self.SF and activation != "relu2") or (shared is not None and activation == "relu2"):
+            raise ValueError("routed experts: shared_ff belongs to relu2 experts, shared to gated ones")
+        self.shared = SwiGLU(hidden_size, **shared) if shared is not None else None
+        self.activation, self.has_correction, self.gated = activation, bool(correction), activation != "relu2"
         self.groups, self.keep, self.route_scale, self.identity = int(groups), int(keep), float(route_scale), int(identity)
         if group_mark not in ("max", "top2_sum"):
             raise ValueError(f"routed experts: group_mark={group_mark!r}")
@@ -80,7 +93,7 @@ class RoutedExperts(FeedForward):
         if self.has_correction:
             s["correction"] = ParamSpec((self.routes,), kind="vector", init="normal")
         for e in range(self.E):
-            if self.activation == "swiglu":
+            if self.gated:
                 s[f"e{e}.gate"] = ParamSpec((self.F, self.hidden))
             s[f"e{e}.up"] = ParamSpec((self.F, self.hidden))
             s[f"e{e}.down"] = ParamSpec((self.hidden, self.F))
@@ -89,19 +102,26 @@ class RoutedExperts(FeedForward):
             s["shared.down"] = ParamSpec((self.hidden, self.SF))
             if self.shared_gate:
                 s["shared.sg"] = ParamSpec((1, self.hidden))
+        if self.shared is not None:
+            s.update({"shared." + n.split("_")[0]: p for n, p in self.shared.param_specs().items()})
         return s
+
+    def attach(self, rt) -> None:
+        super().attach(rt)
+        if self.shared is not None:
+            self.shared.attach(rt)
 
     def bind(self, params: Dict[str, torch.Tensor]) -> None:
         self.w_router = params.pop("router")
         self.up_layout = self.activation
-        if self.activation == "swiglu":
+        if self.gated:
             gates, ups = [params.pop(f"e{e}.gate") for e in range(self.E)], [params.pop(f"e{e}.up") for e in range(self.E)]
             if gates[0].dtype == torch.bfloat16 and self.F % 8 == 0 and self.hidden % 8 == 0 and hasattr(self.rt.k, "moe_grouped"):
                 # an expert's first matrix in sixteens of 8 gate rows and the 8 matching up rows: the layout whose
-                # product writes silu(gate) * up from its epilogue
+                # product writes the activation from its epilogue
                 from ..kernels import interleave_gate_up
                 self.w_up = torch.stack([interleave_gate_up(g, u) for g, u in zip(gates, ups)]).contiguous()
-                self.up_layout = "swiglu_interleaved"
+                self.up_layout = self.activation + "_interleaved"
             else:
                 # its gate rows, then its up rows
                 self.w_up = torch.stack([torch.cat([g, u]) for g, u in zip(gates, ups)]).contiguous()
@@ -115,6 +135,8 @@ class RoutedExperts(FeedForward):
             self.w_sup, self.w_sdown = params.pop("shared.up"), params.pop("shared.down")
             self.w_sg = params.pop("shared.sg") if self.shared_gate else None
             self.check_products(shared_up=self.w_sup, shared_down=self.w_sdown)
+        if self.shared is not None:
+            self.shared.bind({f"{n}_proj.weight": params.pop("shared." + n) for n in ("gate", "up", "down")})
         # bfloat16: the router's logits (and the shared gate's) as one product of the library with fp32 sums and fp32
         # output (bf16 operands multiply exactly in fp32); the 32-bit path keeps the FFMA router kernel
         self.w_route = None
@@ -127,10 +149,10 @@ class RoutedExperts(FeedForward):
         if self.has_correction:
             out["correction"] = self.correction
         for e in range(self.E):
-            if self.up_layout == "swiglu_interleaved":
+            if self.up_layout.endswith("_interleaved"):
                 gu = self.w_up[e].view(self.F // 8, 2, 8, self.hidden)
                 out[f"e{e}.gate"], out[f"e{e}.up"] = gu[:, 0].reshape(self.F, self.hidden), gu[:, 1].reshape(self.F, self.hidden)
-            elif self.activation == "swiglu":
+            elif self.gated:
                 out[f"e{e}.gate"], out[f"e{e}.up"] = self.w_up[e, :self.F], self.w_up[e, self.F:]
             else:
                 out[f"e{e}.up"] = self.w_up[e]
@@ -139,6 +161,8 @@ class RoutedExperts(FeedForward):
             out["shared.up"], out["shared.down"] = self.w_sup, self.w_sdown
             if self.shared_gate:
                 out["shared.sg"] = self.w_sg
+        if self.shared is not None:
+            out.update({"shared." + n.split("_")[0]: t for n, t in self.shared.tensors().items()})
         return out
 
     def forward(self, x: torch.Tensor, residual: torch.Tensor, ctx: StepContext) -> None:
@@ -155,16 +179,20 @@ class RoutedExperts(FeedForward):
         else:
             k.moe_route(idx, wgt, x, self.w_router, self.top, gate, self.w_sg, self.score, self.renormalize,
                         self.correction, self.groups, self.keep, self.route_scale, self.group_top)
-        grouped = self.up_layout == "swiglu_interleaved" or (self.activation == "relu2" and not self.identity)
+        if self.shared is not None:
+            # ahead of the routed experts: where the stream counts as zeros its last product then stores
+            self.shared.forward(x, residual, ctx)
+        clamp = {"limit": self.limit, "alpha": self.alpha} if self.activation == "swish_limit" else {}
+        grouped = self.up_layout.endswith("_interleaved") or (self.activation == "relu2" and not self.identity)
         if (grouped and T > 16 and rt.dtype == torch.bfloat16 and self.F % 8 == 0 and self.hidden % 8 == 0
                 and x.stride(0) % 8 == 0 and hasattr(k, "moe_grouped")):
             # many tokens: pairs sorted by expert, each expert's rows as tiles of one grouped product
             k.moe_grouped(residual, x, self.w_up, self.w_down, idx, wgt, self.scale_input,
-                          activation=self.up_layout, identity=bool(self.identity))
+                          activation=self.up_layout, identity=bool(self.identity), **clamp)
         else:
             # few tokens (and the 32-bit path): every (token, choice) streams its expert's matrices
             act = rt.ws.get("moe.act", (T, self.top, self.F), rt.dtype)
-            k.moe_up(act, x, self.w_up, idx, wgt, self.scale_input, self.up_layout)
+            k.moe_up(act, x, self.w_up, idx, wgt, self.scale_input, self.up_layout, **clamp)
             k.moe_down(residual, act, self.w_down, idx, x if self.identity else None, wgt)
         if self.SF:
             u = rt.ws.get("moe.shared_u", (T, self.SF), rt.dtype)

@@ -5,7 +5,8 @@ y = (x * 1/sqrt(mean(x^2) + eps)) * w, weight used as it is
 row (a tensor without dimensions) instead of a weight per coordinate.  ``layer_scale``: a second vector ``scale``
 multiplies the normed row coordinate by coordinate (a layer's learned scale on its sublayer's output).
 ``one_plus``: the checkpoint stores the weight around zero and the row is multiplied by 1 + w (the sum is made once,
-in fp32, when the weights are bound).
+in fp32, when the weights are bound).  ``multiplier``: a constant on the whole normed row (a residual multiplier; made
+part of the fp32 weight when that is bound).
 """
 from __future__ import annotations
 
@@ -21,9 +22,10 @@ from .base import Norm, ParamSpec
 class RMSNorm(Norm):
     reads_stream_by_kernel = True
 
-    def __init__(self, size: int, eps: float, scalar: bool = False, layer_scale: bool = False, one_plus: bool = False):
+    def __init__(self, size: int, eps: float, scalar: bool = False, layer_scale: bool = False, one_plus: bool = False,
+                 multiplier: float = 1.0):
         self.size = int(size)
-        self.one_plus = bool(one_plus)
+        self.one_plus, self.multiplier = bool(one_plus), float(multiplier)
         self.stored: Optional[torch.Tensor] = None
         self.eps = float(eps)
         self.scalar = bool(scalar)
@@ -42,18 +44,21 @@ class RMSNorm(Norm):
 
     def bind(self, params: Dict[str, torch.Tensor]) -> None:
         self.weight = params["weight"]
-        if self.one_plus:
+        if self.one_plus or self.multiplier != 1.0:
             self.stored = self.weight
-            self.weight = (1.0 + self.stored.float()).contiguous()
+            self.weight = self.stored.float()
+            if self.one_plus:
+                self.weight = 1.0 + self.weight
+            self.weight = (self.weight * self.multiplier).contiguous()
         self.scale = params.get("scale")
         if self.scalar:
             # the kernels (and the products that fold a norm in) read a weight per coordinate: the one
             # gain, widened to 32 bits (exact), repeated along the row
-            self.gain = self.stored if self.one_plus else self.weight
+            self.gain = self.stored if self.stored is not None else self.weight
             self.weight = self.weight.float().reshape(1).expand(self.size).contiguous()
 
     def tensors(self) -> Dict[str, torch.Tensor]:
-        out = {"weight": self.gain if self.scalar else (self.stored if self.one_plus else self.weight)}
+        out = {"weight": self.gain if self.scalar else (self.stored if self.stored is not None else self.weight)}
         if self.layer_scale:
             out["scale"] = self.scale
         return out

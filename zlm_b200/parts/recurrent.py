@@ -1,4 +1,4 @@
-"""Three recurrent mixers whose whole memory of a sequence is a fixed-size fp32 state.
+"""Four recurrent mixers whose whole memory of a sequence is a fixed-size fp32 state.
 
 ``rglru``: a recurrent block with a real-gated linear recurrent unit.  Two branches of ``width`` channels read the
 mixer's input:
@@ -25,7 +25,18 @@ The state per sequence is S [heads, head_dim, v_dim] fp32.
     z = sigmoid(W_z x + b_z),  u = W_x x + b_x,  cand = u + 1/2 where u >= 0, sigmoid(u) where u < 0
     S_t = (1 - z) S_(t-1) + z cand,  out = W_o (S * silu(W_g x))
 
-The state per sequence is S [width] fp32.  In all of them everything between the projections and the output
+The state per sequence is S [width] fp32.
+
+``mlstm``: a matrix memory with exponential gates and a running maximum that keeps them in range, per head:
+
+    q = W_q x * head_dim^-1/2, k = W_k x, v = W_v x                          heads x head_dim, heads x v_dim
+    i = cap tanh((W_i x + b_i) / cap),  f = log sigmoid(cap tanh((W_f x + b_f) / cap))
+    m_t = max(f + m_(t-1), i)                                                m starts at 0
+    S_t = exp(f + m_(t-1) - m_t) S_(t-1) + exp(i - m_t) k_t v_t^T,  n_t likewise with k_t alone
+    o_t = S_t^T q_t / (max(|n_t . q_t|, exp(-m_t)) + 1e-6)
+    out = W_o (rms_norm_per_head(o) * w_norm * sigmoid(W_g x))               w_norm [heads * v_dim]
+
+The state per sequence is S [heads, head_dim, v_dim], n [heads, head_dim] and m [heads], fp32.  In all of them everything between the projections and the output
 projection's input is fp32 whatever the compute dtype.
 """
 from __future__ import annotations
@@ -197,3 +208,82 @@ class MinGRU(Mixer):
             gated[:, W:].zero_()
         k.mingru(gated[:, :W], proj, 0, W, 2 * W, self.b_z, self.b_x, io.state, ctx)
         k.linear(residual, gated, self.w_o, accumulate=True, defer=True)       # a norm reads the stream next
+
+
+@register_mixer("mlstm")
+class MatrixLSTM(Mixer):
+    reads_input_by_products = True       # x goes into the fused projections and nowhere else
+
+    def __init__(self, hidden_size: int, num_heads: int, head_dim: int, v_dim: int, gate_cap: float, norm_eps: float):
+        """``gate_cap`` 0: the gates' logits are not capped."""
+        self.hidden = int(hidden_size)
+        self.H, self.D, self.V = int(num_heads), int(head_dim), int(v_dim)
+        self.cap, self.eps = float(gate_cap), float(norm_eps)
+        if min(self.H, self.D, self.V) <= 0 or self.cap < 0:
+            raise ValueError(f"mlstm: {self.H} heads of {self.D} / {self.V}, gates capped at {self.cap}")
+        self.QK, self.VV = self.H * self.D, self.H * self.V
+
+    def param_specs(self) -> Dict[str, ParamSpec]:
+        K = self.hidden
+        s = {"q_proj.weight": ParamSpec((self.QK, K)), "k_proj.weight": ParamSpec((self.QK, K)),
+             "v_proj.weight": ParamSpec((self.VV, K)), "g_proj.weight": ParamSpec((self.VV, K)),
+             "norm.weight": ParamSpec((self.VV,), kind="vector", init="one_plus_normal"),
+             "o_proj.weight": ParamSpec((K, self.VV))}
+        for n in ("i", "f"):
+            s[f"{n}_gate.weight"] = ParamSpec((self.H, K))
+            s[f"{n}_gate.bias"] = ParamSpec((self.H,), kind="vector", init="zeros")
+        return s
+
+    def state_request(self):
+        return (StateRequest((self.H, self.D, self.V), torch.float32), StateRequest((self.H, self.D), torch.float32),
+                StateRequest((self.H,), torch.float32))
+
+    def bind(self, params: Dict[str, torch.Tensor]) -> None:
+        # one fused projection: rows [q | k | v | g | i | f], with rows of zeros up to a multiple of 8; the gates' rows also
+        # by themselves, for steps of many tokens: their logits are fp32 whatever the compute dtype
+        rows = [params.pop(f"{n}_proj.weight") for n in ("q", "k", "v", "g")] + [params.pop(f"{n}_gate.weight") for n in ("i", "f")]
+        self.N = 2 * self.QK + 2 * self.VV
+        extra = -(self.N + 2 * self.H) % 8
+        if extra:
+            rows.append(torch.zeros((extra, self.hidden), dtype=rows[0].dtype, device=rows[0].device))
+        self.w_in = torch.cat(rows, dim=0).contiguous()
+        self.b_i, self.b_f = params.pop("i_gate.bias"), params.pop("f_gate.bias")
+        if self.b_i.dtype != self.b_f.dtype:
+            self.b_i, self.b_f = self.b_i.float(), self.b_f.float()
+        self.w_norm = params.pop("norm.weight")
+        self.w_o = pad_inner(params.pop("o_proj.weight"))
+        self.check_products(in_proj=self.w_in, o_proj=self.w_o)
+
+    def tensors(self) -> Dict[str, torch.Tensor]:
+        a, b, c, d, H = self.QK, 2 * self.QK, 2 * self.QK + self.VV, self.N, self.H
+        return {"q_proj.weight": self.w_in[:a], "k_proj.weight": self.w_in[a:b], "v_proj.weight": self.w_in[b:c],
+                "g_proj.weight": self.w_in[c:d], "i_gate.weight": self.w_in[d:d + H], "f_gate.weight": self.w_in[d + H:d + 2 * H],
+                "i_gate.bias": self.b_i, "f_gate.bias": self.b_f, "norm.weight": self.w_norm, "o_proj.weight": self.w_o[:, :self.VV]}
+
+    def forward(self, x: torch.Tensor, residual: torch.Tensor, ctx: StepContext, io: LayerIO) -> None:
+        rt, k = self.rt, self.rt.k
+        T, H, D, V, N, VV = x.shape[0], self.H, self.D, self.V, self.N, self.VV
+        q_off, k_off, v_off, g_off = 0, self.QK, 2 * self.QK, 2 * self.QK + VV
+        step = ctx.is_decode and ctx.T == ctx.R
+        if rt.dtype == torch.float32 or (step and T <= 16):
+            # (few tokens: one product with fp32 outputs serves the gates too)
+            proj = rt.ws.get("mlstm.proj", (T, self.w_in.shape[0]), torch.float32)
+            k.linear(proj, x, self.w_in)
+            z, i_off = proj, N
+        else:
+            proj = rt.ws.get("mlstm.proj", (T, N), rt.dtype)
+            k.linear(proj, x, self.w_in[:N])
+            z, i_off = rt.ws.get("mlstm.gates", (T, self.w_in.shape[0] - N), torch.float32), 0
+            k.linear(z, x, self.w_in[N:])
+        cols = self.w_o.shape[1]
+        y = rt.ws.get("mlstm.gated", (T, cols), rt.dtype)
+        if cols > VV:
+            y[:, VV:].zero_()
+        gates = (z, i_off, i_off + H, self.b_i, self.b_f, self.cap, io.state, ctx, H, D, V, D ** -0.5)
+        if step:
+            k.mlstm_step(y[:, :VV], proj, q_off, k_off, v_off, g_off, *gates, self.w_norm, self.eps)
+        else:
+            o = rt.ws.get("mlstm.o", (T, VV), torch.float32)
+            k.mlstm(o, proj, q_off, k_off, v_off, *gates)
+            k.norm_gate(y[:, :VV], o, proj[:, g_off:g_off + VV], H, V, "head", self.w_norm, self.eps, "sigmoid")
+        k.linear(residual, y, self.w_o, accumulate=True, defer=True)       # a norm reads the stream next

@@ -74,12 +74,19 @@ class RotaryInterleaved(PositionEncoding):
     """Rotary encoding on neighbouring pairs (2i, 2i + 1), i < dims / 2: the pair is turned by
     pos * base^(-2i / dims); what lies beyond ``dims`` in the rotated vector passes unchanged.  The
     part carries the table of frequencies (computed in 64-bit, rounded to fp32); the mixer's own
-    kernel forms the angle, its sine and cosine in fp32."""
+    kernel forms the angle, its sine and cosine in fp32.
+
+    ``scaling`` ({"factor", "original", "low", "high"}): frequencies for contexts longer than the ``original`` one, by
+    their wavelength l = 2 pi / f: as they are where l < original / high, divided by ``factor`` where l > original / low,
+    and between the two (1 - s) f / factor + s f with s = (original / l - low) / (high - low)."""
     fused = True
     interleaved = True
 
-    def __init__(self, base: float, dims: int):
+    def __init__(self, base: float, dims: int, scaling: Optional[Mapping[str, Any]] = None):
         self.base = float(base)
+        self.scaling = None if scaling is None else {k: float(scaling[k]) for k in ("factor", "original", "low", "high")}
+        if self.scaling is not None and min(self.scaling.values()) <= 0:
+            raise ValueError(f"rope: frequencies scaled by {self.scaling}")
         self.n_rot = int(dims)
         if self.n_rot % 2 or self.n_rot < 0:
             raise ValueError(f"rope: dims={self.n_rot} must be even")
@@ -89,6 +96,13 @@ class RotaryInterleaved(PositionEncoding):
         super().attach(rt)
         i = torch.arange(self.n_rot // 2, dtype=torch.float64)
         inv = torch.pow(torch.tensor(self.base, dtype=torch.float64), -2.0 * i / max(self.n_rot, 1))
+        if self.scaling is not None:
+            sc = self.scaling
+            length = 2.0 * math.pi / inv
+            s = (sc["original"] / length - sc["low"]) / (sc["high"] - sc["low"]) if sc["high"] != sc["low"] else torch.ones_like(inv)
+            mixed = (1.0 - s) * inv / sc["factor"] + s * inv
+            inv = torch.where(length < sc["original"] / sc["high"], inv,
+                              torch.where(length > sc["original"] / sc["low"], inv / sc["factor"], mixed))
         self.inv_freq = inv.to(torch.float32).to(rt.device)
 
 
