@@ -4,7 +4,8 @@ package's kernels, cache and scheduler with it.
 
 A model is (config, tensors): ``config`` is the design's config.json as a dict, ``tensors`` maps checkpoint names to
 torch tensors.  ``forward(config, tensors, tokens)`` returns (logits [T, vocab], stream after every layer
-[layers, T, width], every token's closest routing call).
+[layers, T, width], every token's closest routing call, how much is left of every token's memory read-outs after
+cancellation).
 """
 from __future__ import annotations
 
@@ -160,10 +161,16 @@ def attention_2(h, p: str, c: Mapping, tensors, eps: float, first) -> torch.Tens
 
 
 # ---------------------------------------------------------------------------------------------- matrix memory
-def matrix_memory(q, k, v, i, f, start_max: float = 0.0) -> torch.Tensor:
-    """q, k [T, H, D], v [T, H, V], log gates i, f [T, H] -> [T, H, V], token by token with the running maximum."""
+def empty_memory(H: int, D: int, V: int):
+    return torch.zeros(H, D, V, dtype=F64), torch.zeros(H, D, dtype=F64), torch.zeros(H, dtype=F64)
+
+
+def matrix_memory(q, k, v, i, f, state=None, left=None):
+    """q, k [T, H, D], v [T, H, V], log gates i, f [T, H] -> ([T, H, V], the state after them), token by token with the
+    running maximum; ``state`` (S, n, m): where to start, nothing and a maximum of 0 if not given.  ``left`` [T] is lowered
+    to |S^T q| / sum_d |S_d| |q_d|, the smallest of the heads': where that is tiny, the read-out is what rounding leaves."""
     T, H, D = q.shape
-    S, n, m = torch.zeros(H, D, v.shape[2], dtype=F64), torch.zeros(H, D, dtype=F64), torch.full((H,), start_max, dtype=F64)
+    S, n, m = state if state is not None else empty_memory(H, D, v.shape[2])
     out = torch.zeros(T, H, v.shape[2], dtype=F64)
     for t in range(T):
         m_new = torch.maximum(f[t] + m, i[t])
@@ -172,8 +179,11 @@ def matrix_memory(q, k, v, i, f, start_max: float = 0.0) -> torch.Tensor:
         n = keep[:, None] * n + take[:, None] * k[t]
         m = m_new
         den = torch.maximum((n * q[t]).sum(-1).abs(), torch.exp(-m)) + 1e-6
-        out[t] = torch.einsum("hdv,hd->hv", S, q[t]) / den[:, None]
-    return out
+        read = torch.einsum("hdv,hd->hv", S, q[t])
+        out[t] = read / den[:, None]
+        if left is not None:
+            left[t] = torch.minimum(left[t], (read.norm(dim=-1) / (S.norm(dim=-1) * q[t].abs()).sum(-1).clamp_min(1e-30)).min())
+    return out, (S, n, m)
 
 
 def memory_gates(h, p: str, c: Mapping, tensors) -> Tuple[torch.Tensor, torch.Tensor]:
@@ -183,14 +193,14 @@ def memory_gates(h, p: str, c: Mapping, tensors) -> Tuple[torch.Tensor, torch.Te
     return i, f
 
 
-def mlstm(h, p: str, c: Mapping, tensors, eps: float) -> torch.Tensor:
+def mlstm(h, p: str, c: Mapping, tensors, eps: float, left=None) -> torch.Tensor:
     T = h.shape[0]
     H, D, V = int(c["heads"]), int(c["dim"]), int(c["vdim"])
     q = (h @ _w(tensors, p + "q").T).view(T, H, D) * D ** -0.5
     k = (h @ _w(tensors, p + "k").T).view(T, H, D)
     v = (h @ _w(tensors, p + "v").T).view(T, H, V)
     i, f = memory_gates(h, p, c, tensors)
-    o = rms_norm(matrix_memory(q, k, v, i, f), None, eps).reshape(T, H * V)
+    o = rms_norm(matrix_memory(q, k, v, i, f, left=left)[0], None, eps).reshape(T, H * V)
     return (o * _w(tensors, p + "norm") * torch.sigmoid(h @ _w(tensors, p + "g").T)) @ _w(tensors, p + "o").T
 
 
@@ -243,6 +253,7 @@ def forward(config: Mapping, tensors: Mapping[str, torch.Tensor], tokens, tilt: 
     eps, m = float(config["norm"]["eps"]), float(config.get("residual_mult", 1.0))
     x = _w(tensors, "embed")[torch.as_tensor(list(tokens), dtype=torch.long)]
     margin = torch.full((x.shape[0],), math.inf, dtype=F64)
+    left = torch.ones(x.shape[0], dtype=F64)
     first: Dict[str, torch.Tensor] = {}
     layers = []
     for i, l in enumerate(config["layers"]):
@@ -252,7 +263,7 @@ def forward(config: Mapping, tensors: Mapping[str, torch.Tensor], tokens, tilt: 
         elif l["type"] == "attention_2":
             y = attention_2(x, p + "mix.", c, tensors, eps, first)
         elif l["type"] == "mlstm":
-            y = mlstm(x, p + "mix.", c, tensors, eps)
+            y = mlstm(x, p + "mix.", c, tensors, eps, left)
         else:
             raise ValueError(l["type"])
         x = x + m * rms_norm(y, _w(tensors, p + "norm1"), eps)
@@ -265,4 +276,4 @@ def forward(config: Mapping, tensors: Mapping[str, torch.Tensor], tokens, tilt: 
             x = x + m * rms_norm(y, _w(tensors, p + "norm2"), eps)
         layers.append(x)
     logits = rms_norm(x, _w(tensors, "final.norm"), eps) @ _w(tensors, "head").T
-    return logits, torch.stack(layers), margin
+    return logits, torch.stack(layers), margin, left

@@ -87,11 +87,12 @@ class CacheGroup:
 
     def __init__(self, request: CacheRequest, entries: List[int], num_pages: int, num_slots: int,
                  max_pages_per_slot: int, dtype: torch.dtype, device, stager: Optional[TableStager] = None,
-                 reach: Sequence[Tuple[int, int, int]] = ()):
-        """``reach``: (window, chunk, first keys kept) of every entry that reads this group's cache, its own entries among them (empty:
-        the request's)."""
+                 reach: Sequence[Tuple[int, int]] = (), keep: int = 0):
+        """``reach``: (window, chunk) of every entry that reads this group's cache, its own entries among them (empty:
+        the request's); ``keep``: the most first keys of a sequence that any of them reads beside its window."""
         self.request = request
-        self.reach = tuple(reach) or ((request.window, request.chunk, request.keep),)
+        self.reach = tuple(reach) or ((request.window, request.chunk),)
+        self.keep = max(int(keep), request.keep)
         self.stager = stager
         self.entries = entries
         self.num_pages = num_pages
@@ -138,13 +139,12 @@ class CacheGroup:
         def first(window: int, chunk: int) -> int:
             lo = max(0, length + 1 - window) if window else 0
             return max(lo, length - length % chunk) if chunk else lo
-        first_needed = min(first(w, c) for w, c, _ in self.reach)
-        kept = pages_for(max(k for _, _, k in self.reach))
+        first_needed = min(first(w, c) for w, c in self.reach)
         if first_needed < PAGE_TOKENS:
             return
         have = self.slot_pages.get(slot, [])
         back = []
-        for lp in range(kept, min(len(have), first_needed // PAGE_TOKENS)):
+        for lp in range(pages_for(self.keep), min(len(have), first_needed // PAGE_TOKENS)):
             if have[lp] >= 0:
                 back.append(have[lp])
                 have[lp] = -1
@@ -183,18 +183,20 @@ class KVCache:
         # groups by request, over the entries that keep a cache of their own, and by how far back their readers look
         # (an entry that reads another one's cache has a window of its own: the pages stay as long as either needs them)
         readers: Dict[int, set] = {}
+        keeps: Dict[int, int] = {}
         for i, (e, r) in enumerate(zip(schedule, requests)):
             if r is not None:
-                readers.setdefault(i if e.cache_of is None else e.cache_of, set()).add((r.window, r.chunk, r.keep))
+                readers.setdefault(i if e.cache_of is None else e.cache_of, set()).add((r.window, r.chunk))
+                keeps[i if e.cache_of is None else e.cache_of] = max(keeps.get(i if e.cache_of is None else e.cache_of, 0), r.keep)
         by_req: Dict[Tuple, List[int]] = {}
         for i, (e, r) in enumerate(zip(schedule, requests)):
             if r is not None and e.cache_of is None:
-                by_req.setdefault((r, tuple(sorted(readers[i]))), []).append(i)
+                by_req.setdefault((r, tuple(sorted(readers[i])), keeps[i]), []).append(i)
         self.table_stager = TableStager(self.num_pages * max(1, len(by_req)), device)
         self.groups: List[CacheGroup] = [
             CacheGroup(r, ents, self.num_pages, self.max_slots, max_pages_per_slot, dtype, device,
-                       self.table_stager, reach)
-            for (r, reach), ents in by_req.items()]
+                       self.table_stager, reach, keep)
+            for (r, reach, keep), ents in by_req.items()]
         where: Dict[int, Tuple[CacheGroup, int]] = {}
         for g in self.groups:
             for j, ent in enumerate(g.entries):

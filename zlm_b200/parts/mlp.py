@@ -39,32 +39,37 @@ class SwiGLU(FeedForward):
                 "down_proj.weight": ParamSpec((self.hidden, self.inter))}
 
     def bind(self, params: Dict[str, torch.Tensor]) -> None:
-        gate, up = params.pop("gate_proj.weight"), params.pop("up_proj.weight")
+        gate, up, down = params.pop("gate_proj.weight"), params.pop("up_proj.weight"), params.pop("down_proj.weight")
+        # bf16: channels of zeros up to a multiple of 8 (act(0) * 0 = 0 in every form): what the products read at a time
+        self.cols = self.inter + (-self.inter % 8 if gate.dtype == torch.bfloat16 else 0)
+        if self.cols > self.inter:
+            more = (0, 0, 0, self.cols - self.inter)
+            gate, up, down = torch.nn.functional.pad(gate, more), torch.nn.functional.pad(up, more), pad_inner(down)
         # bf16: gate and up rows interleaved in eights, so that the product's epilogue holds
         # a channel's gate and up together and writes act(gate) * up directly
-        self.fused = (gate.dtype == torch.bfloat16 and self.inter % 8 == 0 and hasattr(self.rt.k, "linear_swiglu")
+        self.fused = (gate.dtype == torch.bfloat16 and hasattr(self.rt.k, "linear_swiglu")
                       and (self.act == "silu" or getattr(self.rt.k, "gated_activations", ()).count(self.act)))
         if self.fused:
             from ..kernels import interleave_gate_up
             self.w_gu = interleave_gate_up(gate, up)
         else:
             self.w_gu = torch.cat([gate, up], dim=0).contiguous()
-        self.w_down = params.pop("down_proj.weight")
+        self.w_down = down
         self.check_products(gate_up_proj=self.w_gu, down_proj=self.w_down)
 
     def tensors(self) -> Dict[str, torch.Tensor]:
-        I, K = self.inter, self.hidden
+        I, K, n = self.cols, self.hidden, self.inter
         if self.fused:
             gu = self.w_gu.view(I // 8, 2, 8, K)
             gate, up = gu[:, 0].reshape(I, K), gu[:, 1].reshape(I, K)
         else:
             gate, up = self.w_gu[:I], self.w_gu[I:]
-        return {"gate_proj.weight": gate, "up_proj.weight": up, "down_proj.weight": self.w_down}
+        return {"gate_proj.weight": gate[:n], "up_proj.weight": up[:n], "down_proj.weight": self.w_down[:, :n]}
 
     def forward(self, x: torch.Tensor, residual: torch.Tensor, ctx: StepContext) -> None:
         rt, k = self.rt, self.rt.k
         T = x.shape[0]
-        act = rt.ws.get("ffn.act", (T, self.inter), rt.dtype)
+        act = rt.ws.get("ffn.act", (T, self.cols), rt.dtype)
         if self.fused:
             if self.act == "silu":
                 k.linear_swiglu(act, x, self.w_gu)
@@ -73,7 +78,7 @@ class SwiGLU(FeedForward):
             else:
                 k.linear_swiglu(act, x, self.w_gu, act=self.act)
         else:
-            gu = rt.ws.get("ffn.gu", (T, 2 * self.inter), rt.dtype)
+            gu = rt.ws.get("ffn.gu", (T, 2 * self.cols), rt.dtype)
             k.linear(gu, x, self.w_gu)
             if self.act == "silu":
                 k.swiglu(act, gu)

@@ -114,9 +114,16 @@ class RoutedExperts(FeedForward):
     def bind(self, params: Dict[str, torch.Tensor]) -> None:
         self.w_router = params.pop("router")
         self.up_layout = self.activation
+        self.cols = self.F                        # an expert's channels, with the padding
         if self.gated:
             gates, ups = [params.pop(f"e{e}.gate") for e in range(self.E)], [params.pop(f"e{e}.up") for e in range(self.E)]
-            if gates[0].dtype == torch.bfloat16 and self.F % 8 == 0 and self.hidden % 8 == 0 and hasattr(self.rt.k, "moe_grouped"):
+            # bf16: channels of zeros up to a multiple of 8 (act(0) * 0 = 0 in both forms)
+            extra = -self.F % 8 if gates[0].dtype == torch.bfloat16 else 0
+            if extra:
+                gates, ups = ([torch.nn.functional.pad(t, (0, 0, 0, extra)) for t in ts] for ts in (gates, ups))
+                params.update({f"e{e}.down": torch.nn.functional.pad(params[f"e{e}.down"], (0, extra)) for e in range(self.E)})
+                self.cols = self.F + extra
+            if gates[0].dtype == torch.bfloat16 and self.hidden % 8 == 0 and hasattr(self.rt.k, "moe_grouped"):
                 # an expert's first matrix in sixteens of 8 gate rows and the 8 matching up rows: the layout whose
                 # product writes the activation from its epilogue
                 from ..kernels import interleave_gate_up
@@ -150,13 +157,13 @@ class RoutedExperts(FeedForward):
             out["correction"] = self.correction
         for e in range(self.E):
             if self.up_layout.endswith("_interleaved"):
-                gu = self.w_up[e].view(self.F // 8, 2, 8, self.hidden)
-                out[f"e{e}.gate"], out[f"e{e}.up"] = gu[:, 0].reshape(self.F, self.hidden), gu[:, 1].reshape(self.F, self.hidden)
+                gu = self.w_up[e].view(self.cols // 8, 2, 8, self.hidden)
+                out[f"e{e}.gate"], out[f"e{e}.up"] = (gu[:, x].reshape(self.cols, self.hidden)[:self.F] for x in (0, 1))
             elif self.gated:
-                out[f"e{e}.gate"], out[f"e{e}.up"] = self.w_up[e, :self.F], self.w_up[e, self.F:]
+                out[f"e{e}.gate"], out[f"e{e}.up"] = self.w_up[e, :self.F], self.w_up[e, self.cols:self.cols + self.F]
             else:
                 out[f"e{e}.up"] = self.w_up[e]
-            out[f"e{e}.down"] = self.w_down[e]
+            out[f"e{e}.down"] = self.w_down[e, :, :self.F]
         if self.SF:
             out["shared.up"], out["shared.down"] = self.w_sup, self.w_sdown
             if self.shared_gate:
@@ -184,14 +191,14 @@ class RoutedExperts(FeedForward):
             self.shared.forward(x, residual, ctx)
         clamp = {"limit": self.limit, "alpha": self.alpha} if self.activation == "swish_limit" else {}
         grouped = self.up_layout.endswith("_interleaved") or (self.activation == "relu2" and not self.identity)
-        if (grouped and T > 16 and rt.dtype == torch.bfloat16 and self.F % 8 == 0 and self.hidden % 8 == 0
+        if (grouped and T > 16 and rt.dtype == torch.bfloat16 and self.cols % 8 == 0 and self.hidden % 8 == 0
                 and x.stride(0) % 8 == 0 and hasattr(k, "moe_grouped")):
             # many tokens: pairs sorted by expert, each expert's rows as tiles of one grouped product
             k.moe_grouped(residual, x, self.w_up, self.w_down, idx, wgt, self.scale_input,
                           activation=self.up_layout, identity=bool(self.identity), **clamp)
         else:
             # few tokens (and the 32-bit path): every (token, choice) streams its expert's matrices
-            act = rt.ws.get("moe.act", (T, self.top, self.F), rt.dtype)
+            act = rt.ws.get("moe.act", (T, self.top, self.cols), rt.dtype)
             k.moe_up(act, x, self.w_up, idx, wgt, self.scale_input, self.up_layout, **clamp)
             k.moe_down(residual, act, self.w_down, idx, x if self.identity else None, wgt)
         if self.SF:
