@@ -654,9 +654,37 @@ MURILIX_SIZES = {
     "wide": (_murilix(4096, 32, 128, 64, 128, 1536, 512, 4096, 4096, 18432, 32, 2, 2048, 4, 256, "gLlg", 32768),
              _nuvilorn_twin(4096, 32, 128, 64, 128, 512, 18432, 32, 2, 2048, "LLlL", 32768)),
 }
+def _lolivik(width, heads, kv_heads, window, keep, ff, experts, top, expert_ff, kinds, vocab):
+    """Layers of kind "a" (every earlier token, a bias by distance up to 512), "w" (a window and the first tokens, rotation)
+    and "m" (a matrix memory of 128 x 128 a head); heads of 128 throughout; the first layer's feed-forward dense, the others
+    routed, with a shared expert as wide as a routed one."""
+    sizes = {"heads": heads, "kv_heads": kv_heads, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "v_mix": True}
+    mix = {"a": dict(sizes, softcap=30.0, bias_max=512, q_temp={"coef": 0.1, "every": 1024}),
+           "w": dict(sizes, mask={"size": window, "keep_first": keep},
+                     rot={"base": 500000.0, "dims": 64, "scaling": {"factor": 8.0, "original": 8192, "low": 1.0, "high": 4.0}}),
+           "m": {"heads": heads, "dim": 128, "vdim": 128, "gate_cap": 15.0}}
+    kind = {"a": "attention", "w": "attention_2", "m": "mlstm"}
+    moe = {"kind": "moe", "expert": {"ff": expert_ff, "limit": 7.0}, "router": {"experts": experts, "top": top},
+           "shared": {"ff": expert_ff, "limit": 7.0}}
+    return {"architecture": "Lolivik", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "residual_mult": 0.5,
+            "layers": [{"type": kind[k], "mixer": mix[k], "mlp": {"kind": "dense", "ff": ff} if i == 0 else moe}
+                       for i, k in enumerate(kinds)]}
+
+
+# Lolivik beside Zekazen at the same width, heads, layers, vocabulary and experts: retention (128 x 128 a head) where Lolivik
+# has a matrix memory, attention behind convolutions where it has either attention, and one more expert a token instead of
+# the shared one.  Windows that cover the run, or a quarter of it ("small": Lolivik's alone, in its "w" layers)
+LOLIVIK_SIZES = {
+    "lite": (_lolivik(2048, 16, 4, 4096, 64, 5120, 32, 4, 1024, "amwmaw", 32768),
+             _zekazen(2048, 16, 4, 4096, 32, 0, 5, 1024, 8, 4, "araraa", 32768)),
+    "small": (_lolivik(1024, 8, 2, 512, 64, 2560, 16, 4, 512, "amwmaw", 32768),
+              _zekazen(1024, 8, 2, 4096, 16, 0, 5, 512, 4, 2, "araraa", 32768)),
+    "wide": (_lolivik(4096, 32, 8, 4096, 64, 6144, 16, 2, 2048, "amwm", 32768),
+             _zekazen(4096, 32, 8, 4096, 16, 0, 3, 2048, 4, 2, "arar", 32768)),
+}
 DESIGNS = {"nuvilorn": ("Nuvilorn", DESIGN_SIZES), "zekazen": ("Zekazen", ZEKAZEN_SIZES),
            "lodevik": ("Lodevik", LODEVIK_SIZES), "sudupel": ("Sudupel", SUDUPEL_SIZES),
-           "murilix": ("Murilix", MURILIX_SIZES)}
+           "murilix": ("Murilix", MURILIX_SIZES), "lolivik": ("Lolivik", LOLIVIK_SIZES)}
 
 
 def design_comparison(args) -> int:
@@ -673,8 +701,8 @@ def design_comparison(args) -> int:
     B, L, steps, warmup = args.batch, PROMPT_LEN, min(args.steps, 64), max(3, args.warmup)
     g = torch.Generator().manual_seed(0)
     design, sizes = DESIGNS[args.design]
-    twin = "qwen3_twin" if "architectures" in next(iter(sizes.values()))[1] else "nuvilorn_twin"
-    beside = {"qwen3_twin": "Qwen3 dense", "nuvilorn_twin": "Nuvilorn"}[twin]
+    beside = next(iter(sizes.values()))[1].get("architecture", "Qwen3 dense")
+    twin = "qwen3_twin" if beside == "Qwen3 dense" else beside.lower() + "_twin"
     out = {"metric": f"prefill and decode tokens/s of {design} beside {beside} at equal sizes", "unit": "tokens/s",
            "dtype": "bf16", "data": "synthetic", "batch": B, "prompt_len": L, "peaks": pk, "sizes": {}}
     for name in ([args.design_size] if args.design_size else list(sizes)):

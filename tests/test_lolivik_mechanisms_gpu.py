@@ -75,7 +75,7 @@ def plan_for(lens, starts, slots):
 def attend_in_pages(dtype, H, G, hd, vd, lens, starts, impl=None, **opt):
     """The attention kernel on sequences whose keys and values lie in shuffled pages (whatever a query must not read is
     there too, and pages that no query may touch hold NaN), against the plain attention; -> (got, want) per sequence."""
-    from zlm_b200.kernels import PAGE_TOKENS, get_kernels
+    from zlm_b200.kernels import PAGE_TOKENS, get_kernels, pad_bias
     k = get_kernels()
     dt = torch_dtype(dtype)
     g = torch.Generator().manual_seed(H * 1000 + hd + sum(lens))
@@ -112,7 +112,7 @@ def attend_in_pages(dtype, H, G, hd, vd, lens, starts, impl=None, **opt):
     sinks, bias = opt.get("sinks"), opt.get("bias")
     k.attention(out, q_new, pool.to(dt).cuda(), table.cuda(), plan.token_pos, plan.token_slot, H, G, hd, scale, window, plan,
                 v_dim=vd if vd < hd else None, softcap=opt.get("softcap", 0.0), keep=keep,
-                sinks=None if sinks is None else sinks.cuda(), bias=None if bias is None else bias.cuda())
+                sinks=None if sinks is None else sinks.cuda(), bias=None if bias is None else pad_bias(bias).cuda())
     got = out.cpu().view(plan.T, H, hd)
     assert vd == hd or float(got[..., vd:].float().abs().max()) == 0.0
     pairs, at = [], 0

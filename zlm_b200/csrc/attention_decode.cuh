@@ -109,11 +109,25 @@ __device__ __forceinline__ void attention_decode_item(
         if (qd == 0) l0 = l1 = 1.f;
     }
 
+    const float* const b0 = attn_bias_row(opt, kvh * G + min(g, G - 1));           // (rows beyond the group hold nothing that counts)
+    const float* const b1 = attn_bias_row(opt, kvh * G + min(g + 8, G - 1));
     for (int p = p_begin; p < p_end; ++p) {
         const int stage = (p - p_begin) & 1;
+        const int kbase = walk.page(p) * ZLM_PAGE + warp * 16;
+        // the page's biases are on their way while the page is waited for
+        float bz[2][4] = {};
+        if (opt.bias) {
+#pragma unroll
+            for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+                for (int e = 0; e < 2; ++e) {
+                    const int n = min(pos - (kbase + nt * 8 + qd * 2 + e), opt.bias_n - 1);
+                    bz[nt][e] = attn_bias_at(b0, n);
+                    if (G > 8) bz[nt][2 + e] = attn_bias_at(b1, n);
+                }
+        }
         dec_wait<1>();                       // everything but the newest group has landed: page p is there
         gs.sync();
-        const int kbase = walk.page(p) * ZLM_PAGE + warp * 16;
         const bool busy = !(kbase > pos || (kbase + 15 < t_start && kbase >= opt.keep));       // warp-uniform
         if (busy) {
         const __nv_bfloat16* kt = Ks + stage * TILE;
@@ -137,17 +151,11 @@ __device__ __forceinline__ void attention_decode_item(
         // scale (to base-2 exponent) and mask by position
         float mx0 = -INFINITY, mx1 = -INFINITY;
         attn_scores_log2<2>(s, scale_log2, softcap);
-        if (opt.bias) {                                // (rows beyond the group hold nothing that counts)
-            const float* b0 = opt.bias + (size_t)(kvh * G + min(g, G - 1)) * opt.bias_n;
-            const float* b1 = opt.bias + (size_t)(kvh * G + min(g + 8, G - 1)) * opt.bias_n;
+        if (opt.bias) {
 #pragma unroll
             for (int nt = 0; nt < 2; ++nt)
 #pragma unroll
-                for (int e = 0; e < 2; ++e) {
-                    const int n = pos - (kbase + nt * 8 + qd * 2 + e);
-                    s[nt][e] += attn_bias_log2(b0, n, opt.bias_n);
-                    if (G > 8) s[nt][2 + e] += attn_bias_log2(b1, n, opt.bias_n);
-                }
+                for (int e = 0; e < 4; ++e) s[nt][e] = fmaf(bz[nt][e], ATTN_LOG2E, s[nt][e]);
         }
 #pragma unroll
         for (int nt = 0; nt < 2; ++nt)

@@ -14,7 +14,7 @@
 // joins the softmax's denominator without a value; without the array the flag `sink` stands for a 0), and
 // `v_share` (that many neighbouring key heads read one value head: the page is [nkv key heads | nkv / v_share
 // value heads] of [ZLM_PAGE][hd] each), `keep` (with a window: the sequence's first `keep` keys stay visible) and `bias`
-// ([nq][bias_n], added after the cap by distance, the last entry for all greater distances).
+// (bias_n numbers a head, added after the cap by distance, the last one for all greater distances; attn_common.cuh).
 #include "common.cuh"
 #include "attn_common.cuh"
 
@@ -65,7 +65,7 @@ attention_generic_kernel(TA* __restrict__ out, int out_stride, const TA* __restr
 
     const int c0 = t_start / 32, c1 = pos / 32;
     const int kept = keep > 0 ? min((keep - 1) / 32 + 1, c0) : 0;         // chunks of the first kept keys ahead of the window's
-    const float* brow = bias ? bias + (size_t)h * bias_n : nullptr;
+    const float* brow = attn_bias_row(AttnOpts{chunk, softcap, sinks, v_share, keep, bias, bias_n}, h);
     for (int c = warp; c <= c1; c += ATT_WARPS) {
         // chunk c holds keys [32c, 32c+32); chunk c belongs to warp c % ATT_WARPS
         if (c >= kept && c < c0) {                 // between the kept keys and the window: on to this warp's first chunk there
@@ -87,7 +87,7 @@ attention_generic_kernel(TA* __restrict__ out, int out_stride, const TA* __restr
             for (int e = 0; e < hd; ++e) d = fmaf(qs[e], to_f32(kr[e]), d);
             s = d * scale;
             if (softcap > 0.f) s = softcap * tanhf(s / softcap);
-            if (brow && ZLM_CHK(brow + min(pos - key, bias_n - 1), 4)) s += brow[min(pos - key, bias_n - 1)];
+            if (brow) s += attn_bias_at(brow, min(pos - key, bias_n - 1));
         }
         const float cm = warp_max(s);          // the chunk holds at least one valid key
         const float mn = fmaxf(m, cm);

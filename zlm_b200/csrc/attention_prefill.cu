@@ -74,8 +74,8 @@ attention_prefill_kernel(__nv_bfloat16* __restrict__ out, int out_stride, const 
     const int blk_lo = attn_first_key(blk_first, window, chunk);
     const AttnWalk walk(blk_lo / ZLM_PAGE, blk_last / ZLM_PAGE + 1, opt.keep);
     const int keep = opt.keep;
-    const float* brow = opt.bias ? opt.bias + (size_t)head * opt.bias_n : nullptr;
-    const float far_bias = brow ? attn_bias_log2(brow, opt.bias_n, opt.bias_n) : 0.f;
+    const float* brow = attn_bias_row(opt, head);
+    const float far_bias = brow ? attn_bias_at(brow, opt.bias_n - 1) * ATTN_LOG2E : 0.f;
     const int w_first = start + row0 + warp * 16;
     const int w_last = min(blk_last, w_first + 15);
     const int w_lo = attn_first_key(w_first, window, chunk);
@@ -162,8 +162,8 @@ attention_prefill_kernel(__nv_bfloat16* __restrict__ out, int out_stride, const 
 #pragma unroll
                 for (int e = 0; e < 2; ++e) {
                     const int key = kbase + nt * 8 + qd * 2 + e;
-                    s[nt][e] += far ? far_bias : attn_bias_log2(brow, pos0 - key, opt.bias_n);
-                    s[nt][2 + e] += far ? far_bias : attn_bias_log2(brow, pos1 - key, opt.bias_n);
+                    s[nt][e] = far ? s[nt][e] + far_bias : fmaf(attn_bias_at(brow, pos0 - key), ATTN_LOG2E, s[nt][e]);
+                    s[nt][2 + e] = far ? s[nt][2 + e] + far_bias : fmaf(attn_bias_at(brow, pos1 - key), ATTN_LOG2E, s[nt][2 + e]);
                 }
         }
 #pragma unroll

@@ -344,8 +344,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         float m_ref = sink ? attn_sink_log2(opt.sinks, head) : -INFINITY, l = sink ? 1.f : 0.f;
         constexpr bool capped = CAP;
         const int keep = KEEP ? opt.keep : 0;
-        const float* brow = BIAS ? opt.bias + (size_t)head * opt.bias_n : nullptr;
-        const float far_bias = BIAS ? attn_bias_log2(brow, opt.bias_n, opt.bias_n) : 0.f;
+        const float* brow = BIAS ? attn_bias_row(opt, head) : nullptr;
+        const float far_bias = BIAS ? attn_bias_at(brow, opt.bias_n - 1) * ATTN_LOG2E : 0.f;
         const float k_in = capped ? 2.0f * scale_log2 / opt.softcap : 0.f, k_out = opt.softcap * 1.4426950408889634f;
         bool ok = true;
         for (int j = 0; j < NS; ++j) {
@@ -364,17 +364,19 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             tc_fence_before();
             __syncwarp();
             if (lane == 0) mbar_arrive(&s_empty[hh]);
-            // a bias that differs from key to key goes into the scores before their maximum: they are then final base-2
-            // exponents; the scores of a step whose distances all read the table's last entry stay raw
+            // with a bias the scores become base-2 exponents before their maximum is taken (scaled and capped here, not
+            // below); where the step's distances all read the table's last number, that one is part of the reference
             const bool near = BIAS && first_pos - (kb1 + ZLM_PAGE - 1) < opt.bias_n - 1;        // block-uniform
-            if (near) {
+            if (BIAS) {
 #pragma unroll
-                for (int e = 0; e < FA_BK; ++e) {
-                    const int key = kb0 + e;
-                    sv[e] = (capped ? fa_cap(sv[e], k_in, k_out) : sv[e] * scale_log2) + attn_bias_log2(brow, pos - key, opt.bias_n);
+                for (int e = 0; e < FA_BK; ++e) sv[e] = capped ? fa_cap(sv[e], k_in, k_out) : sv[e] * scale_log2;
+                if (near) {
+#pragma unroll
+                    for (int e = 0; e < FA_BK; ++e)       // (neighbouring rows read neighbouring numbers)
+                        sv[e] = fmaf(attn_bias_at(brow + (pos - kb0), -e), ATTN_LOG2E, sv[e]);
                 }
             }
-            // four independent chains of maxima (raw scores, unless the bias went in; the scale is positive)
+            // four independent chains of maxima (raw scores without a bias; the scale is positive)
             float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
             if (inner) {
 #pragma unroll
@@ -390,7 +392,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             }
             // (the cap is monotonic too: the capped maximum is the maximum's cap)
             const float mx_raw = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
-            const float mx = near ? mx_raw : (capped ? fa_cap(mx_raw, k_in, k_out) : mx_raw * scale_log2) + (BIAS ? far_bias : 0.f);          // -inf stays -inf
+            const float mx = BIAS ? mx_raw + (near ? 0.f : far_bias) : capped ? fa_cap(mx_raw, k_in, k_out) : mx_raw * scale_log2;          // -inf stays -inf
             // lazy reference: move it only when the maximum grew by more than 2^8
             const bool grow = mx > m_ref + FA_RESCALE;              // also true for the first real maximum
             const float m_new = grow ? mx : m_ref;
@@ -426,7 +428,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                 float p[8];
 #pragma unroll
                 for (int e = 0; e < 8; ++e) {
-                    p[e] = near ? fa_ex2(sv[ch * 8 + e] - ref)
+                    p[e] = BIAS ? fa_ex2(sv[ch * 8 + e] - ref)
                          : capped ? fa_ex2(fa_cap(sv[ch * 8 + e], k_in, k_out) - ref)
                                   : fa_ex2(fmaf(sv[ch * 8 + e], scale_log2, -ref));
                     ps4[e & 3] += p[e];

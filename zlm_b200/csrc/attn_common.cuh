@@ -41,8 +41,10 @@ __device__ __forceinline__ unsigned pack_bf16(float lo, float hi) {
 //   v_share  that many neighbouring key heads read one value head: a page is [nkv key heads | nkv / v_share value
 //            heads] of [ZLM_PAGE][hd] each (1: the ordinary [K | V] of nkv heads each)
 //   keep     > 0 (with a window): the sequence's first `keep` positions stay visible beside the window
-//   bias     numbers [nq][bias_n] added to the scores after scale and cap, by distance: query i reads
-//            bias[head][min(i - j, bias_n - 1)] for key j
+//   bias     numbers added to the scores after scale and cap, by distance: bias_n of them a head, query i reads the
+//            min(i - j, bias_n - 1)-th for key j.  A head's row of the table is [ATTN_BIAS_LEAD | bias_n | ATTN_BIAS_TAIL]
+//            floats: what comes before the first number is never used, what follows repeats the last one, so that a tile
+//            with a distance below bias_n - 1 in it reads the table at pos - key for all its keys, seen or not
 struct AttnOpts {
     int chunk;
     float softcap;
@@ -84,29 +86,28 @@ struct AttnWalk {
 // whether the query at `pos` whose window starts at `lo` reads the key
 __device__ __forceinline__ bool attn_sees(int key, int pos, int lo, int keep) { return key <= pos && (key >= lo || key < keep); }
 
-// the bias of a head (its row of the table) at a distance, in base-2 exponents
-__device__ __forceinline__ float attn_bias_log2(const float* row, int distance, int bias_n) {
-    const float* p = row + min(max(distance, 0), bias_n - 1);
-    return ZLM_CHK(p, 4) ? __ldg(p) * ATTN_LOG2E : 0.f;
+#define ATTN_BIAS_LEAD 256
+#define ATTN_BIAS_TAIL 256
+// a head's bias at distance 0 in the table (null: no bias)
+__device__ __forceinline__ const float* attn_bias_row(const AttnOpts& opt, int head) {
+    return opt.bias ? opt.bias + (size_t)head * (ATTN_BIAS_LEAD + opt.bias_n + ATTN_BIAS_TAIL) + ATTN_BIAS_LEAD : nullptr;
+}
+// the bias at a distance between -ATTN_BIAS_LEAD and bias_n - 1 + ATTN_BIAS_TAIL
+__device__ __forceinline__ float attn_bias_at(const float* row, int distance) {
+    return ZLM_CHK(row + distance, 4) ? __ldg(row + distance) : 0.f;
 }
 
-// a raw dot product as a base-2 exponent: dot * scale * log2(e), capped first where the mixer asks for it
-// (tanh through one exponential: 1 - 2 / (e^{2x} + 1), absolute error of a few 1e-7 of the cap)
-__device__ __forceinline__ float attn_score_log2(float dot, float scale_log2, float softcap) {
-    if (softcap <= 0.f) return dot * scale_log2;
-    const float x = dot * scale_log2 / softcap;               // y = dot * scale / softcap = x / log2(e): e^{2y} = 2^{2x}
-    const float th = 1.0f - __fdividef(2.0f, exp2f(2.0f * x) + 1.0f);
-    return softcap * 1.4426950408889634f * th;
-}
-
-// a tile's raw dot products as base-2 exponents, all at once: whether there is a cap is asked once (every thread of
-// a launch answers alike), so a kernel without one pays a multiplication a score and nothing else
+// a tile's raw dot products as base-2 exponents, dot * scale * log2(e), capped first where the mixer asks for it (tanh(y)
+// through one exponential: 1 - 2 / (e^{2y} + 1), absolute error of a few 1e-7 of the cap).  Whether there is a cap is asked
+// once for the tile (every thread of a launch answers alike), so a kernel without one pays a multiplication a score and
+// nothing else
 template <int NT> __device__ __forceinline__ void attn_scores_log2(float (&s)[NT][4], float scale_log2, float softcap) {
     if (softcap > 0.f) {
+        const float k_in = 2.0f * scale_log2 / softcap, k_out = softcap * ATTN_LOG2E;         // 2^(dot * k_in) = e^{2y}
 #pragma unroll
         for (int nt = 0; nt < NT; ++nt)
 #pragma unroll
-            for (int e = 0; e < 4; ++e) s[nt][e] = attn_score_log2(s[nt][e], scale_log2, softcap);
+            for (int e = 0; e < 4; ++e) s[nt][e] = fmaf(-2.0f * k_out, __fdividef(1.0f, exp2f(s[nt][e] * k_in) + 1.0f), k_out);
     } else {
 #pragma unroll
         for (int nt = 0; nt < NT; ++nt)

@@ -24,8 +24,19 @@ GATED_LIMIT = 8          # g sigmoid(alpha g) (u + 1) on clamped halves; its two
 GATED_GELU = 7      # as SWIGLU with gelu_tanh(gate) instead of silu(gate)
 
 
+# floats beside a head's numbers in a bias table (attn_common.cuh)
+BIAS_LEAD, BIAS_TAIL = 256, 256
+
+
 class KernelError(RuntimeError):
     pass
+
+
+def pad_bias(bias: torch.Tensor) -> torch.Tensor:
+    """[heads, BIAS_LEAD + n + BIAS_TAIL] fp32 from the biases [heads, n] of the distances 0 .. n - 1: the layout that
+    ``attention`` reads (the first number repeated in front, the last one behind)."""
+    b = bias.float()
+    return torch.cat([b[:, :1].expand(-1, BIAS_LEAD), b, b[:, -1:].expand(-1, BIAS_TAIL)], dim=1).contiguous()
 
 
 def interleave_gate_up(gate: torch.Tensor, up: torch.Tensor) -> torch.Tensor:
@@ -714,13 +725,14 @@ class CudaKernels:
         ``softcap``: scores become softcap * tanh(score / softcap) after the scale.  ``v_share``: that many
         neighbouring key heads read one value head; a page of the pool is then [nkv key heads | nkv / v_share
         value heads] of [PAGE_TOKENS, hd] each (with 1, the ordinary [2, nkv, PAGE_TOKENS, hd]).  ``keep``: with a
-        window, the sequence's first ``keep`` keys stay visible beside it.  ``bias`` [nq, n] fp32: added to the scores
-        after scale and cap, bias[h, min(distance, n - 1)]."""
+        window, the sequence's first ``keep`` keys stay visible beside it.  ``bias``: ``pad_bias`` of numbers b [nq, n] that
+        are added to the scores after scale and cap, b[h, min(distance, n - 1)]."""
         T = q.shape[0]
         bias_n = 0
         if bias is not None:
             assert bias.dtype == torch.float32 and bias.dim() == 2 and bias.shape[0] == nq and bias.is_contiguous()
-            bias_n = int(bias.shape[1])
+            bias_n = int(bias.shape[1]) - BIAS_LEAD - BIAS_TAIL
+            assert bias_n > 0
         assert keep >= 0 and (keep == 0 or (window > 0 and not chunk))
         if sinks is not None:
             assert sinks.dtype == torch.float32 and sinks.shape == (nq,) and sinks.is_contiguous()

@@ -34,7 +34,7 @@ from typing import Any, Dict, List, Mapping, Optional, Union
 
 import torch
 
-from ..kernels import PAGE_TOKENS
+from ..kernels import PAGE_TOKENS, pad_bias
 from ..registry import POSITION_ENCODINGS, lookup, register_mixer
 from .base import CacheRequest, LayerIO, Mixer, ParamSpec, StateRequest, StepContext
 
@@ -167,7 +167,7 @@ class ConvAttention(Mixer):
             if table.shape[0] // 2 >= self.far and table.shape[0] > 1:
                 raise ValueError(f"attention: a distance bias of {table.shape[0]} rows up to a distance of {self.far}")
             rows = torch.tensor(distance_rows(table.shape[0], self.far), device=table.device)
-            self.bias = table.float()[rows].t().contiguous()
+            self.bias = pad_bias(table.float()[rows].t())
         if self.learned_sink:
             self.sinks = self.stored["sinks"].float().contiguous()
         self.lam = float(self.stored["v_mix"].float()) if self.v_mix == "reader" else 0.0

@@ -28,6 +28,8 @@ from typing import Dict, List, Optional, Sequence, Tuple
 
 import torch
 
+from .parts.base import Part
+
 
 @dataclass
 class OpRecord:
@@ -181,7 +183,7 @@ class ProfilingKernels:
                            n_rot, token_pos, token_slot, block_table, pool, nq, nkv, hd, write)
 
     @staticmethod
-    def _reach(plan, window: int, chunk: int):
+    def _reach(plan, window: int, chunk: int, keep: int = 0):
         """(keys the step reads of the cache, query-key pairs it scores) from the step's host-side plan."""
         def first(p):
             lo = max(0, p + 1 - window) if window else 0
@@ -190,22 +192,23 @@ class ProfilingKernels:
         if plan is not None and getattr(plan, "h_seq_start", None):
             for start, new in zip(plan.h_seq_start, plan.h_seq_new):
                 end = start + new
-                keys_read += end - first(start)
+                keys_read += end - first(start) + min(keep, first(start))
                 for p in range(start, end):                 # visible keys of each new token
-                    pairs += (p + 1) - first(p)
+                    pairs += (p + 1) - first(p) + min(keep, first(p))
         return keys_read, pairs
 
     def attention(self, out, q, pool, block_table, token_pos, token_slot, nq, nkv, hd, scale, window, plan=None,
-                  len_bucket=None, v_dim=None, sink=False, chunk=0, v_share=1, **kw):
+                  len_bucket=None, v_dim=None, sink=False, chunk=0, v_share=1, keep=0, bias=None, **kw):
         T, el = q.shape[0], q.element_size()
-        keys_read, pairs = self._reach(plan, window, chunk)
+        keys_read, pairs = self._reach(plan, window, chunk, keep)
         n = 2 * T * nq * hd * el + keys_read * (nkv + nkv // v_share) * hd * pool.element_size()
         kind = "attention decode" if (plan is not None and plan.is_decode) else "attention prefill"
         if v_share > 1:
             kind += ", %d maps on one value head" % v_share
+        kind += (", bias by distance" if bias is not None else "") + (", first tokens kept" if keep else "")
         return self._timed(kind, n, 2.0 * nq * (hd + (v_dim or hd)) * pairs, self.k.attention, out, q, pool, block_table,
                            token_pos, token_slot, nq, nkv, hd, scale, window, plan, len_bucket=len_bucket, v_dim=v_dim,
-                           sink=sink, chunk=chunk, v_share=v_share, **kw)
+                           sink=sink, chunk=chunk, v_share=v_share, keep=keep, bias=bias, **kw)
 
     # differential attention and the stream of designs that norm a sublayer's output
     def diff_prep(self, q_out, proj, *args, **kw):
@@ -285,6 +288,19 @@ class ProfilingKernels:
         kind = "gated linear attention decode" if plan.is_decode else "gated linear attention prefill"
         return self._timed(kind, n, 6.0 * T * heads * dim * v_dim, self.k.linear_attention, o, proj, q_off, k_off, v_off,
                            alpha, head_decay, state, plan, heads, dim, v_dim, *args, **kw)
+
+    def mlstm(self, o, proj, q_off, k_off, v_off, z, i_off, f_off, b_i, b_f, cap, state, plan, heads, dim, v_dim, *args):
+        T, el = proj.shape[0], proj.element_size()
+        n = T * heads * (2 * dim + v_dim) * el + _nbytes(o) + 2 * plan.R * heads * dim * v_dim * 4
+        # (fp32 multiply-adds on the ordinary cores: state update and read-out, as for the other recurrences)
+        return self._timed("matrix memory prefill", n, 4.0 * T * heads * dim * v_dim, self.k.mlstm, o, proj, q_off, k_off, v_off, z,
+                           i_off, f_off, b_i, b_f, cap, state, plan, heads, dim, v_dim, *args)
+
+    def mlstm_step(self, out, proj, q_off, k_off, v_off, g_off, z, i_off, f_off, b_i, b_f, cap, state, plan, heads, dim, v_dim, *args):
+        T, el = proj.shape[0], proj.element_size()
+        n = T * heads * 2 * (dim + v_dim) * el + _nbytes(out) + 2 * plan.R * heads * dim * v_dim * 4
+        return self._timed("matrix memory decode (norm and gate with it)", n, 4.0 * T * heads * dim * v_dim, self.k.mlstm_step, out,
+                           proj, q_off, k_off, v_off, g_off, z, i_off, f_off, b_i, b_f, cap, state, plan, heads, dim, v_dim, *args)
 
     def norm_add_norm(self, stream, y, w1, eps1, out2, w2, eps2, center=False, conv=None):
         n, name = 3 * _nbytes(stream) + _nbytes(out2), "sublayer norm+add+next norm"
@@ -372,10 +388,10 @@ class ProfilingKernels:
     def _experts_read(self, T, top, w):
         return min(T * top, w.shape[0]) * w.shape[1] * w.shape[2] * w.element_size()
 
-    def moe_up(self, act, x, w_up, idx, wgt, scale_input=True, activation="relu2"):
+    def moe_up(self, act, x, w_up, idx, wgt, scale_input=True, activation="relu2", **kw):
         T, top = idx.shape
         return self._timed("experts up", self._experts_read(T, top, w_up) + _nbytes(act), 2.0 * T * top * w_up.shape[1] * w_up.shape[2],
-                           self.k.moe_up, act, x, w_up, idx, wgt, scale_input, activation)
+                           self.k.moe_up, act, x, w_up, idx, wgt, scale_input, activation, **kw)
 
     def moe_down(self, stream, act, w_down, idx, identity_input=None, wgt=None):
         T, top = idx.shape
@@ -383,7 +399,8 @@ class ProfilingKernels:
                            2.0 * T * top * w_down.shape[1] * w_down.shape[2], self.k.moe_down, stream, act, w_down, idx,
                            identity_input, wgt)
 
-    def moe_grouped(self, stream, x, w_up, w_down, idx, wgt, scale_input=True, impl=None, activation="relu2", identity=False):
+    def moe_grouped(self, stream, x, w_up, w_down, idx, wgt, scale_input=True, impl=None, activation="relu2", identity=False,
+                    **kw):
         T, top = idx.shape
         n = self._experts_read(T, top, w_up) + self._experts_read(T, top, w_down) + 2 * _nbytes(stream) + T * top * (
             4 * w_up.shape[1] + 8 * w_down.shape[1] + 2 * x.shape[1])
@@ -391,7 +408,7 @@ class ProfilingKernels:
         return self._timed("experts (sorted, grouped up+down)", n,
                            2.0 * T * top * (w_up.shape[1] * w_up.shape[2] + w_down.shape[1] * w_down.shape[2]),
                            self.k.moe_grouped, stream, x, w_up, w_down, idx, wgt, scale_input, impl=impl,
-                           activation=activation, identity=identity)
+                           activation=activation, identity=identity, **kw)
 
     def relu2_scale(self, out, u, row_scale=None):
         return self._timed("relu2*gate", _nbytes(out) + _nbytes(u), 0, self.k.relu2_scale, out, u, row_scale)
@@ -412,6 +429,7 @@ def weight_names(model) -> Dict[int, str]:
         children = getattr(b, "children", None)
         if children:
             parts += list(children().values())
+    parts += [p.shared for p in parts if isinstance(getattr(p, "shared", None), Part)]        # (a part inside another)
     for p in parts:
         for attr, val in vars(p).items():
             if isinstance(val, torch.Tensor) and val.dim() == 2 and val.is_cuda:
