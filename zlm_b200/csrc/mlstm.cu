@@ -62,41 +62,46 @@ template <int VEC> __device__ __forceinline__ void ml_store(float* p, const MlVe
 // ---------------------------------------------------------------------------- one token a sequence
 // grid (R * cluster, H), clusters along x; a block owns the columns [rank * VC, ...) of one head of one sequence.  A thread
 // owns VEC neighbouring columns of every RG-th row.
-#define ML_AHEAD 8
+#define ML_AHEAD 4
 template <typename TA, typename TO, int VEC>
-__global__ void __launch_bounds__(ML_THREADS)
+__global__ void __launch_bounds__(ML_THREADS, 4)
 mlstm_step_kernel(TO* __restrict__ out, int out_stride, const TA* __restrict__ proj, int stride, int q_off, int k_off, int v_off,
                   int g_off, MlstmGates gates, float* __restrict__ S, float* __restrict__ nvec, float* __restrict__ mmax,
                   const int* __restrict__ seq_slot, const int* __restrict__ cu_seqlens, int H, int D, int V, int VC, float q_scale,
                   VecW w_norm, float eps) {
     cg::cluster_group cluster = cg::this_cluster();
-    extern __shared__ __align__(16) float ml_smem[];       // q [D], k [D], new n [D], sums [RG][VC], o [VC]
+    extern __shared__ __align__(16) float ml_smem[];       // q [D], k [D], new n [D], sums [rows][VC], o [VC]
     __shared__ float red[32];
     __shared__ float squares;
     const int NS = cluster.num_blocks(), rank = cluster.block_rank();
     const int r = blockIdx.x / NS, h = blockIdx.y, tid = threadIdx.x;
     const int CG = VC / VEC, RG = ML_THREADS / CG;
     const int rg = tid / CG, cc = (tid - rg * CG) * VEC;
+    const bool folds = 32 % CG == 0 && RG * CG == ML_THREADS;      // a warp holds whole rows: their sums meet in shuffles first
+    const int rows = folds ? ML_THREADS / 32 : RG;
     const int c0 = rank * VC, ncol = max(0, min(VC, V - c0));
     const bool live = rg < RG && cc < ncol;
     float* sq = ml_smem;
     float* sk = sq + D;
     float* sn = sk + D;
     float* sums = sn + D;
-    float* so = sums + RG * VC;
+    float* so = sums + rows * VC;
     const bool ok = ZLM_CHK(seq_slot + r, 4) && ZLM_CHK(cu_seqlens + r, 4);      // (block-uniform; the cluster's barriers below are met either way)
     const int slot = ok ? seq_slot[r] : 0;
     const size_t t = ok ? cu_seqlens[r] : 0;
     const size_t sh = (size_t)slot * H + h;
     float* sp = S + (sh * D) * V + c0 + cc;
     // the state is from earlier steps: its first rows are on the way before the wait for the projection
-    MlVec<VEC> first[ML_AHEAD];
+    MlVec<VEC> s[ML_AHEAD];
+    auto load_rows = [&](int d0) {
 #pragma unroll
-    for (int j = 0; j < ML_AHEAD; ++j) {
-        const int d = rg + j * RG;
-        if (live && d < D && ZLM_CHK(sp + (size_t)d * V, VEC * 4)) first[j] = ml_load<VEC>(sp + (size_t)d * V);
-        else memset(&first[j], 0, sizeof(first[j]));
-    }
+        for (int j = 0; j < ML_AHEAD; ++j) {
+            const int d = d0 + j * RG;
+            if (live && d < D && ZLM_CHK(sp + (size_t)d * V, VEC * 4)) s[j] = ml_load<VEC>(sp + (size_t)d * V);
+            else memset(&s[j], 0, sizeof(s[j]));
+        }
+    };
+    load_rows(rg);
     pdl_trigger();
     pdl_wait();
     const TA* row = proj + t * stride;
@@ -124,14 +129,6 @@ mlstm_step_kernel(TO* __restrict__ out, int out_stride, const TA* __restrict__ p
     nq = block_sum(nq, red);                                // (its barriers also publish q, k and n)
     if (live) {
         for (int d0 = rg; d0 < D; d0 += ML_AHEAD * RG) {
-            MlVec<VEC> s[ML_AHEAD];
-#pragma unroll
-            for (int j = 0; j < ML_AHEAD; ++j) {
-                const int d = d0 + j * RG;
-                if (d0 == rg) s[j] = first[j];
-                else if (d < D && ZLM_CHK(sp + (size_t)d * V, VEC * 4)) s[j] = ml_load<VEC>(sp + (size_t)d * V);
-                else memset(&s[j], 0, sizeof(s[j]));
-            }
 #pragma unroll
             for (int j = 0; j < ML_AHEAD; ++j) {
                 const int d = d0 + j * RG;
@@ -144,16 +141,24 @@ mlstm_step_kernel(TO* __restrict__ out, int out_stride, const TA* __restrict__ p
                 }
                 if (ZLM_CHK(sp + (size_t)d * V, VEC * 4)) ml_store<VEC>(sp + (size_t)d * V, s[j]);
             }
+            load_rows(d0 + ML_AHEAD * RG);
         }
+    }
+    if (folds) {
 #pragma unroll
-        for (int e = 0; e < VEC; ++e) sums[rg * VC + cc + e] = acc[e];
+        for (int e = 0; e < VEC; ++e)
+            for (int x = CG; x < 32; x <<= 1) acc[e] += __shfl_xor_sync(0xffffffffu, acc[e], x);
+    }
+    if (live && (!folds || (tid & 31) < CG)) {
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) sums[(folds ? tid >> 5 : rg) * VC + cc + e] = acc[e];
     }
     __syncthreads();
     const float den = ml_denominator(nq, m);
     float ss = 0.f;
     for (int c = tid; c < ncol; c += ML_THREADS) {
         float o = 0.f;
-        for (int x = 0; x < RG; ++x) o += sums[x * VC + c];
+        for (int x = 0; x < rows; ++x) o += sums[x * VC + c];
         o /= den;
         so[c] = o;
         ss = fmaf(o, o, ss);
@@ -225,6 +230,36 @@ __device__ __forceinline__ void ml_load8(const TA* p, int left, bool ok, bool ve
     for (int e = 0; e < 8; ++e) f[e] = (ok && e < left && ZLM_CHK(p + e, sizeof(TA))) ? to_f32(p[e]) : 0.f;
 }
 
+// the same in two steps: fetched as stored, widened later
+template <typename TA> struct MlRaw8 { float v[8]; };
+template <> struct MlRaw8<__nv_bfloat16> { uint4 v; };
+template <typename TA> __device__ __forceinline__ MlRaw8<TA> ml_fetch8(const TA* p, int left, bool ok, bool vec) {
+    MlRaw8<TA> r;
+    if constexpr (sizeof(TA) == 2) {
+        if (ok && vec && left >= 8 && ZLM_CHK(p, 16)) {
+            r.v = *(const uint4*)p;
+        } else {
+            unsigned short h[8];
+#pragma unroll
+            for (int e = 0; e < 8; ++e) h[e] = (ok && e < left && ZLM_CHK(p + e, 2)) ? *(const unsigned short*)(p + e) : (unsigned short)0;
+            r.v = make_uint4(h[0] | (unsigned)h[1] << 16, h[2] | (unsigned)h[3] << 16, h[4] | (unsigned)h[5] << 16, h[6] | (unsigned)h[7] << 16);
+        }
+    } else {
+        ml_load8<TA>(p, left, ok, vec, r.v);
+    }
+    return r;
+}
+__device__ __forceinline__ void ml_widen8(const MlRaw8<float>& r, float* f) {
+#pragma unroll
+    for (int e = 0; e < 8; ++e) f[e] = r.v[e];
+}
+__device__ __forceinline__ void ml_widen8(const MlRaw8<__nv_bfloat16>& r, float* f) {
+    f[0] = __uint_as_float(r.v.x << 16); f[1] = __uint_as_float(r.v.x & 0xffff0000u);
+    f[2] = __uint_as_float(r.v.y << 16); f[3] = __uint_as_float(r.v.y & 0xffff0000u);
+    f[4] = __uint_as_float(r.v.z << 16); f[5] = __uint_as_float(r.v.z & 0xffff0000u);
+    f[6] = __uint_as_float(r.v.w << 16); f[7] = __uint_as_float(r.v.w & 0xffff0000u);
+}
+
 // acc[8][4] += X^T Y over `kn` staged rows: X [kn][ML_LD], the warp's eight columns; Y [kn][ML_COLS], the lane's four
 __device__ __forceinline__ void ml_multiply(float (&acc)[8][4], const float* X, const float* Y, int kn, int warp, int lane) {
 #pragma unroll 4
@@ -275,6 +310,13 @@ mlstm_piece_kernel(float* __restrict__ part, float* __restrict__ part_n, float2*
     MlPiece pc;
     pdl_wait();
     if (!ml_piece(pc, blockIdx.x, H, maxp, seq_slot, cu_seqlens)) return;         // block-uniform
+    // the keys and values are on their way while the gates are worked out
+    float fk[ML_L * 8 / ML_THREADS][8];
+#pragma unroll
+    for (int y = 0; y < ML_L * 8 / ML_THREADS; ++y) {
+        const int x = tid + y * ML_THREADS, l = x / 8, d = (x % 8) * 8;
+        ml_load8<TA>(proj + (size_t)(pc.row0 + l) * stride + k_off + (size_t)pc.h * D + d0 + d, D - d0 - d, l < pc.n, vec, fk[y]);
+    }
     if (warp == 0) {
         const double2 g = ml_piece_gates(gates, pc.row0, pc.n, pc.h, sb, se);
         if (lane == 0) {
@@ -282,7 +324,6 @@ mlstm_piece_kernel(float* __restrict__ part, float* __restrict__ part_n, float2*
             if (blockIdx.y == 0 && blockIdx.z == 0 && ZLM_CHK(part_m + pc.at, 8)) part_m[pc.at] = make_float2((float)g.x, (float)(g.x + g.y));
         }
     }
-    // v while the gates are worked out: four neighbouring columns a thread
     for (int x = tid; x < ML_L * (ML_COLS / 8); x += ML_THREADS) {
         const int l = x / (ML_COLS / 8), c = (x % (ML_COLS / 8)) * 8;
         float f[8];
@@ -291,10 +332,10 @@ mlstm_piece_kernel(float* __restrict__ part, float* __restrict__ part_n, float2*
         *(float4*)(Y + l * ML_COLS + c + 4) = make_float4(f[4], f[5], f[6], f[7]);
     }
     __syncthreads();
-    for (int x = tid; x < ML_L * 8; x += ML_THREADS) {
-        const int l = x / 8, d = (x % 8) * 8;
-        float f[8];
-        ml_load8<TA>(proj + (size_t)(pc.row0 + l) * stride + k_off + (size_t)pc.h * D + d0 + d, D - d0 - d, l < pc.n, vec, f);
+#pragma unroll
+    for (int y = 0; y < ML_L * 8 / ML_THREADS; ++y) {
+        const int x = tid + y * ML_THREADS, l = x / 8, d = (x % 8) * 8;
+        const float* f = fk[y];
         const float w = l < pc.n ? expf((float)(se[l] - top)) : 0.f;
         *(float4*)(X + l * ML_LD + d) = make_float4(f[0] * w, f[1] * w, f[2] * w, f[3] * w);
         *(float4*)(X + l * ML_LD + d + 4) = make_float4(f[4] * w, f[5] * w, f[6] * w, f[7] * w);
@@ -337,7 +378,6 @@ __global__ void __launch_bounds__(128)
 mlstm_chain_kernel(float* __restrict__ part, float* __restrict__ part_n, const float2* __restrict__ part_m, float2* __restrict__ ahead,
                    float* __restrict__ S, float* __restrict__ nvec, const float* __restrict__ mmax, const int* __restrict__ seq_slot,
                    const int* __restrict__ cu_seqlens, int H, int D, int V, int maxp) {
-    __shared__ float2 coef[ML_CHAIN];            // (factor of the state ahead, factor of the piece's own part)
     pdl_launch_dependents();
     const int r = blockIdx.x / H, h = blockIdx.x % H, tid = threadIdx.x;
     pdl_wait();
@@ -348,7 +388,7 @@ mlstm_chain_kernel(float* __restrict__ part, float* __restrict__ part_n, const f
     MlVec<VEC> s;
     memset(&s, 0, sizeof(s));
     if (live) s = ml_load<VEC>(S + sh * DV + e);
-    float m = ZLM_CHK(mmax + sh, 4) ? mmax[sh] : 0.f;      // (thread 0's is the one that counts)
+    float m = ZLM_CHK(mmax + sh, 4) ? mmax[sh] : 0.f;
     const size_t at0 = (size_t)r * maxp * H + h;
     for (int p0 = 0; p0 < np; p0 += ML_CHAIN) {
         const int cnt = min(ML_CHAIN, np - p0);
@@ -359,25 +399,23 @@ mlstm_chain_kernel(float* __restrict__ part, float* __restrict__ part_n, const f
             if (live && j < cnt && ZLM_CHK(src, VEC * 4)) a[j] = ml_load<VEC>(src);
             else memset(&a[j], 0, sizeof(a[j]));
         }
-        __syncthreads();                                    // (the coefficients of the round before have been used)
-        if (tid == 0) {
-            float2 g[ML_CHAIN];
+        // (factor of the state ahead, factor of the piece's own part): every thread works them out for itself
+        float2 coef[ML_CHAIN];
 #pragma unroll
-            for (int j = 0; j < ML_CHAIN; ++j) {
-                const float2* src = part_m + at0 + (size_t)(p0 + j) * H;
-                g[j] = (j < cnt && ZLM_CHK(src, 8)) ? *src : make_float2(0.f, 0.f);
-            }
-#pragma unroll
-            for (int j = 0; j < ML_CHAIN; ++j) {
-                if (j >= cnt) break;
-                const float next = fmaxf(g[j].x + m, g[j].y);
-                coef[j] = make_float2(expf(g[j].x + m - next), expf(g[j].y - next));
-                float2* dst = ahead + at0 + (size_t)(p0 + j) * H;
-                if (blockIdx.y == 0 && ZLM_CHK(dst, 8)) *dst = make_float2(m, next);
-                m = next;
-            }
+        for (int j = 0; j < ML_CHAIN; ++j) {
+            const float2* src = part_m + at0 + (size_t)(p0 + j) * H;
+            coef[j] = (j < cnt && ZLM_CHK(src, 8)) ? *src : make_float2(0.f, 0.f);
         }
-        __syncthreads();
+#pragma unroll
+        for (int j = 0; j < ML_CHAIN; ++j) {
+            if (j >= cnt) break;
+            const float2 g = coef[j];
+            const float next = fmaxf(g.x + m, g.y);
+            coef[j] = make_float2(expf(g.x + m - next), expf(g.y - next));
+            float2* dst = ahead + at0 + (size_t)(p0 + j) * H;
+            if (blockIdx.y == 0 && tid == 0 && ZLM_CHK(dst, 8)) *dst = make_float2(m, next);
+            m = next;
+        }
 #pragma unroll
         for (int j = 0; j < ML_CHAIN; ++j) {
             if (j >= cnt) break;
@@ -392,7 +430,9 @@ mlstm_chain_kernel(float* __restrict__ part, float* __restrict__ part_n, const f
                 float* np_ = nvec + sh * D + d;
                 if (!ZLM_CHK(np_, 4)) continue;
                 float n = *np_;
-                for (int j = 0; j < cnt; ++j) {
+#pragma unroll
+                for (int j = 0; j < ML_CHAIN; ++j) {
+                    if (j >= cnt) break;
                     float* q = part_n + (at0 + (size_t)(p0 + j) * H) * D + d;
                     if (!ZLM_CHK(q, 4)) continue;
                     const float own = *q;
@@ -408,7 +448,7 @@ mlstm_chain_kernel(float* __restrict__ part, float* __restrict__ part_n, const f
 
 // grid (R * maxp * H, ceil(V / 128))
 template <typename TA>
-__global__ void __launch_bounds__(ML_THREADS)
+__global__ void __launch_bounds__(ML_THREADS, 2)
 mlstm_out_kernel(float* __restrict__ o, const TA* __restrict__ proj, int stride, int q_off, int k_off, int v_off, MlstmGates gates,
                  const float* __restrict__ part, const float* __restrict__ part_n, const float2* __restrict__ ahead,
                  float* __restrict__ mmax, const int* __restrict__ seq_slot, const int* __restrict__ cu_seqlens, int H, int D, int V,
@@ -417,7 +457,7 @@ mlstm_out_kernel(float* __restrict__ o, const TA* __restrict__ proj, int stride,
     float* Q = ml_smem;                          // [ML_KC][ML_LD]: 32 coordinates of the tokens' queries
     float* K = Q + ML_KC * ML_LD;                // [ML_KC][ML_LD]: and of their keys
     float* P = K + ML_KC * ML_LD;                // [ML_L keys][ML_LD: tokens]
-    float* Y = P + ML_L * ML_LD;                 // [ML_KC][ML_COLS]: rows of the state ahead, then values
+    float* Y = P + ML_L * ML_LD;                 // [2][ML_KC][ML_COLS]: rows of the state ahead, then values
     __shared__ double sb[ML_L], se[ML_L], sm[ML_L];
     __shared__ float snv[ML_KC];
     pdl_launch_dependents();
@@ -428,6 +468,28 @@ mlstm_out_kernel(float* __restrict__ o, const TA* __restrict__ proj, int stride,
     if (!ml_piece(pc, blockIdx.x, H, maxp, seq_slot, cu_seqlens)) return;         // block-uniform
     if (!ZLM_CHK(ahead + pc.at, 8)) return;
     const float2 ma = ahead[pc.at];
+    // a chunk of 32 coordinates: queries and keys through registers (they are turned round on the way), rows of the state
+    // straight into shared memory; the next chunk is on its way while this one's products run
+    MlRaw8<TA> rq, rk;
+    const int ql = tid & 63, qd = (tid >> 6) * 8;
+    auto fetch = [&](int d0, int buf) {
+        const TA* row = proj + (size_t)(pc.row0 + ql) * stride + (size_t)pc.h * D + d0 + qd;
+        rq = ml_fetch8<TA>(row + q_off, D - d0 - qd, ql < pc.n, vec);
+        rk = ml_fetch8<TA>(row + k_off, D - d0 - qd, ql < pc.n, vec);
+        for (int x = tid; x < ML_KC * (ML_COLS / 4); x += ML_THREADS) {
+            const int d = x / (ML_COLS / 4), c = (x % (ML_COLS / 4)) * 4;
+            const float* src = part + (pc.at * D + d0 + d) * V + c0 + c;
+            float* dst = Y + (size_t)buf * ML_KC * ML_COLS + d * ML_COLS + c;
+            if (d0 + d < D && (V & 3) == 0 && c0 + c < V && ZLM_CHK(src, 16)) {
+                asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"((unsigned)__cvta_generic_to_shared(dst)), "l"(src));
+            } else {
+#pragma unroll
+                for (int e = 0; e < 4; ++e) dst[e] = (d0 + d < D && c0 + c + e < V && ZLM_CHK(src + e, 4)) ? src[e] : 0.f;
+            }
+        }
+        asm volatile("cp.async.commit_group;\n" ::);
+    };
+    fetch(0, 0);
     if (warp == 0) {
         ml_piece_gates(gates, pc.row0, pc.n, pc.h, sb, se);
         __syncwarp();
@@ -456,34 +518,32 @@ mlstm_out_kernel(float* __restrict__ o, const TA* __restrict__ proj, int stride,
 #pragma unroll
         for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
     }
-    for (int d0 = 0; d0 < D; d0 += ML_KC) {
-        __syncthreads();
+    for (int d0 = 0, buf = 0; d0 < D; d0 += ML_KC, buf ^= 1) {
+        __syncthreads();                         // (the products of the chunk before are done)
         {
-            const int l = tid & 63, d = (tid >> 6) * 8;
-            const TA* row = proj + (size_t)(pc.row0 + l) * stride + (size_t)pc.h * D + d0 + d;
             float fq[8], fk[8];
-            ml_load8<TA>(row + q_off, D - d0 - d, l < pc.n, vec, fq);
-            ml_load8<TA>(row + k_off, D - d0 - d, l < pc.n, vec, fk);
+            ml_widen8(rq, fq);
+            ml_widen8(rk, fk);
 #pragma unroll
             for (int x = 0; x < 8; ++x) {
-                Q[(d + x) * ML_LD + l] = fq[x] * q_scale;
-                K[(d + x) * ML_LD + l] = fk[x];
+                Q[(qd + x) * ML_LD + ql] = fq[x] * q_scale;
+                K[(qd + x) * ML_LD + ql] = fk[x];
             }
         }
-        for (int x = tid; x < ML_KC * (ML_COLS / 8); x += ML_THREADS) {
-            const int d = x / (ML_COLS / 8), c = (x % (ML_COLS / 8)) * 8;
-            float f[8];
-            ml_load8<float>(part + (pc.at * D + d0 + d) * V + c0 + c, V - c0 - c, d0 + d < D, (V & 3) == 0, f);
-            *(float4*)(Y + d * ML_COLS + c) = make_float4(f[0], f[1], f[2], f[3]);
-            *(float4*)(Y + d * ML_COLS + c + 4) = make_float4(f[4], f[5], f[6], f[7]);
-        }
         if (tid < ML_KC) snv[tid] = (d0 + tid < D && ZLM_CHK(part_n + pc.at * D + d0 + tid, 4)) ? part_n[pc.at * D + d0 + tid] : 0.f;
+        if (d0 + ML_KC < D) {
+            fetch(d0 + ML_KC, buf ^ 1);
+            asm volatile("cp.async.wait_group 1;\n" ::: "memory");
+        } else {
+            asm volatile("cp.async.wait_group 0;\n" ::: "memory");
+        }
         __syncthreads();
+        const float* Yb = Y + (size_t)buf * ML_KC * ML_COLS;
         const int kn = min(ML_KC, D - d0);
 #pragma unroll 4
         for (int k = 0; k < kn; ++k) {
             const float4 qa = *(const float4*)(Q + k * ML_LD + warp * 8), qb = *(const float4*)(Q + k * ML_LD + warp * 8 + 4);
-            const float4 y = *(const float4*)(Y + k * ML_COLS + lane * 4);
+            const float4 y = *(const float4*)(Yb + k * ML_COLS + lane * 4);
             const float k0 = K[k * ML_LD + lane], k1 = K[k * ML_LD + 32 + lane];            // (a lane's keys: lane and 32 + lane)
             const float q[8] = {qa.x, qa.y, qa.z, qa.w, qb.x, qb.y, qb.z, qb.w};
 #pragma unroll
@@ -625,8 +685,9 @@ extern "C" int zlm_mlstm_step(void* out, int out_stride, int out_dtype, const vo
     int VC;
     const int NS = mlstm_strips(V, vec, &VC);
     ZLM_REQUIRE(VC / vec <= ML_THREADS && (long long)R * NS <= 2147483647LL, "mlstm_step: heads of %d value columns", V);
-    const int RG = ML_THREADS / (VC / vec);
-    const size_t smem = (size_t)(3 * D + RG * VC + VC) * sizeof(float);
+    const int CG = VC / vec, RG = ML_THREADS / CG;
+    const int rows = 32 % CG == 0 && RG * CG == ML_THREADS ? ML_THREADS / 32 : RG;
+    const size_t smem = (size_t)(3 * D + rows * VC + VC) * sizeof(float);
     ZLM_REQUIRE(smem <= 200 * 1024, "mlstm_step: %zu bytes a block", smem);
     const VecW wn{w_norm, w_dtype};
 #define ZLM_ML_STEP(TA, TO)                                                                                                     \
@@ -668,7 +729,7 @@ extern "C" int zlm_mlstm(float* o, const void* proj, int stride, int dtype, int 
     const int vec = (stride * esz) % 16 == 0 && (q_off * esz) % 16 == 0 && (k_off * esz) % 16 == 0 && (v_off * esz) % 16 == 0 &&
                     (D * esz) % 16 == 0 && (V * esz) % 16 == 0 && (uintptr_t)proj % 16 == 0;
     const size_t smem1 = (size_t)ML_L * (ML_LD + ML_COLS) * sizeof(float);
-    const size_t smem3 = (size_t)(2 * ML_KC * ML_LD + ML_L * ML_LD + ML_KC * ML_COLS) * sizeof(float);
+    const size_t smem3 = (size_t)(2 * ML_KC * ML_LD + ML_L * ML_LD + 2 * ML_KC * ML_COLS) * sizeof(float);
     const dim3 g1((unsigned)units, (D + 63) / 64, (V + ML_COLS - 1) / ML_COLS), g3((unsigned)units, (V + ML_COLS - 1) / ML_COLS);
 #define ZLM_ML_RUN(TA)                                                                                                          \
     do {                                                                                                                        \
