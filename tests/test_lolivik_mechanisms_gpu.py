@@ -145,10 +145,10 @@ def check_pairs(pairs, dtype, what):
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("form", sorted(FORMS))
 @pytest.mark.parametrize("step", sorted(STEPS))
-@pytest.mark.parametrize("far,softcap", [(20, 5.0), (300, 0.0), (64, 8.0), (1, 0.0)])
+@pytest.mark.parametrize("far,softcap", [(20, 5.0), (300, 0.0), (64, 8.0), (150, 40.0), (1, 0.0)])
 def test_bias_by_distance_in_every_form(dtype, form, step, far, softcap):
     """A bias of order 2 that differs from distance to distance, alone and with a cap and sinks (which it must not pass
-    through), tables that end inside a tile, beyond the sequences, and after one entry."""
+    through; caps that most scores reach half of, and one that none does), tables that end inside a tile, beyond the sequences, and after one entry."""
     H, G, hd, vd = FORMS[form]
     g = torch.Generator().manual_seed(far)
     bias = 2.0 * torch.randn(H, far + 1, generator=g)

@@ -24,8 +24,8 @@
 // lie beyond every row's position and are masked.  Every wait is bounded (see gemm_tcgen05.cu).
 //
 // Options (AttnOpts, attn_common.cuh): keys of the query's own chunk of positions only; a tanh cap on the scores
-// (tanh through one exponential and one reciprocal of the special-function unit, so a capped step costs the softmax
-// warps three such operations a score instead of one); a sink per query head; several key heads on one value head; the
+// (a series of multiply-adds where a warp's scores of a step are all below half the cap; else tanh through one exponential
+// and one reciprocal of the special-function unit, three such operations a score instead of one); a sink per query head; several key heads on one value head; the
 // sequence's first keys beside a window; a bias by distance (heads of 128 only), read from the table where a step's
 // distances differ and added as one number where they all read its last entry.
 //
@@ -52,11 +52,23 @@ __device__ __forceinline__ float fa_ex2(float x) {
 }
 // a raw score as a capped base-2 exponent: k_out * tanh(y), y = s * scale / softcap, with k_in = 2 * scale *
 // log2(e) / softcap (so that 2^(s * k_in) = e^{2y}) and k_out = softcap * log2(e); tanh(y) = 1 - 2 / (e^{2y} + 1).
-// A masked score (-inf) stays -inf.
 __device__ __forceinline__ float fa_cap(float s, float k_in, float k_out) {
     float r;
     asm("rcp.approx.ftz.f32 %0, %1;\n" : "=f"(r) : "f"(fa_ex2(s * k_in) + 1.0f));
-    return s == -INFINITY ? -INFINITY : fmaf(-2.0f * k_out, r, k_out);
+    return fmaf(-2.0f * k_out, r, k_out);
+}
+// two raw scores with |y| <= 1/2 as capped base-2 exponents: scale_log2 * s * (tanh(y) / y), the quotient by its Taylor
+// series in y^2 (what is left out is below 1e-7); multiply-adds, where the form above keeps the special-function unit busy
+__device__ __forceinline__ float2 fa_cap_small(float2 s, float k_y, float scale_log2) {
+    const float2 y = __fmul2_rn(s, make_float2(k_y, k_y)), x = __fmul2_rn(y, y);
+    float2 p = make_float2(21844.0f / 6081075.0f, 21844.0f / 6081075.0f);
+    p = __ffma2_rn(p, x, make_float2(-1382.0f / 155925.0f, -1382.0f / 155925.0f));
+    p = __ffma2_rn(p, x, make_float2(62.0f / 2835.0f, 62.0f / 2835.0f));
+    p = __ffma2_rn(p, x, make_float2(-17.0f / 315.0f, -17.0f / 315.0f));
+    p = __ffma2_rn(p, x, make_float2(2.0f / 15.0f, 2.0f / 15.0f));
+    p = __ffma2_rn(p, x, make_float2(-1.0f / 3.0f, -1.0f / 3.0f));
+    p = __ffma2_rn(p, x, make_float2(1.0f, 1.0f));
+    return __fmul2_rn(__fmul2_rn(s, make_float2(scale_log2, scale_log2)), p);
 }
 __device__ __forceinline__ unsigned fa_pack(float lo, float hi) {
     __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
@@ -346,7 +358,9 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         const int keep = KEEP ? opt.keep : 0;
         const float* brow = BIAS ? attn_bias_row(opt, head) : nullptr;
         const float far_bias = BIAS ? attn_bias_at(brow, opt.bias_n - 1) * ATTN_LOG2E : 0.f;
-        const float k_in = capped ? 2.0f * scale_log2 / opt.softcap : 0.f, k_out = opt.softcap * 1.4426950408889634f;
+        constexpr bool final_scores = CAP || BIAS;      // the scores become base-2 exponents before their maximum is taken
+        const float k_in = capped ? 2.0f * scale_log2 / opt.softcap : 0.f, k_out = opt.softcap * ATTN_LOG2E;
+        const float k_y = k_in * (0.5f / ATTN_LOG2E);                // y = s * k_y
         bool ok = true;
         for (int j = 0; j < NS; ++j) {
             ok = mbar_wait_warp(&s_full[hh], j & 1, abort_flag, 3);
@@ -364,19 +378,33 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             tc_fence_before();
             __syncwarp();
             if (lane == 0) mbar_arrive(&s_empty[hh]);
-            // with a bias the scores become base-2 exponents before their maximum is taken (scaled and capped here, not
-            // below); where the step's distances all read the table's last number, that one is part of the reference
-            const bool near = BIAS && first_pos - (kb1 + ZLM_PAGE - 1) < opt.bias_n - 1;        // block-uniform
-            if (BIAS) {
+            if (capped) {
+                float am[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
-                for (int e = 0; e < FA_BK; ++e) sv[e] = capped ? fa_cap(sv[e], k_in, k_out) : sv[e] * scale_log2;
-                if (near) {
+                for (int e = 0; e < FA_BK; ++e) am[e & 3] = fmaxf(am[e & 3], fabsf(sv[e]));
+                if (__all_sync(0xffffffffu, fmaxf(fmaxf(am[0], am[1]), fmaxf(am[2], am[3])) * k_y <= 0.5f)) {
 #pragma unroll
-                    for (int e = 0; e < FA_BK; ++e)       // (neighbouring rows read neighbouring numbers)
-                        sv[e] = fmaf(attn_bias_at(brow + (pos - kb0), -e), ATTN_LOG2E, sv[e]);
+                    for (int e = 0; e < FA_BK; e += 2) {
+                        const float2 r = fa_cap_small(make_float2(sv[e], sv[e + 1]), k_y, scale_log2);
+                        sv[e] = r.x;
+                        sv[e + 1] = r.y;
+                    }
+                } else {
+#pragma unroll
+                    for (int e = 0; e < FA_BK; ++e) sv[e] = fa_cap(sv[e], k_in, k_out);
                 }
+            } else if (BIAS) {
+#pragma unroll
+                for (int e = 0; e < FA_BK; ++e) sv[e] *= scale_log2;
             }
-            // four independent chains of maxima (raw scores without a bias; the scale is positive)
+            // (where the step's distances all read the bias table's last number, that one is part of the reference)
+            const bool near = BIAS && first_pos - (kb1 + ZLM_PAGE - 1) < opt.bias_n - 1;        // block-uniform
+            if (near) {
+#pragma unroll
+                for (int e = 0; e < FA_BK; ++e)           // (neighbouring rows read neighbouring numbers)
+                    sv[e] = fmaf(attn_bias_at(brow + (pos - kb0), -e), ATTN_LOG2E, sv[e]);
+            }
+            // four independent chains of maxima (raw scores without cap and bias; the scale is positive)
             float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
             if (inner) {
 #pragma unroll
@@ -390,9 +418,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                     mx4[e & 3] = fmaxf(mx4[e & 3], sv[e]);
                 }
             }
-            // (the cap is monotonic too: the capped maximum is the maximum's cap)
             const float mx_raw = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
-            const float mx = BIAS ? mx_raw + (near ? 0.f : far_bias) : capped ? fa_cap(mx_raw, k_in, k_out) : mx_raw * scale_log2;          // -inf stays -inf
+            const float mx = final_scores ? mx_raw + (BIAS && !near ? far_bias : 0.f) : mx_raw * scale_log2;          // -inf stays -inf
             // lazy reference: move it only when the maximum grew by more than 2^8
             const bool grow = mx > m_ref + FA_RESCALE;              // also true for the first real maximum
             const float m_new = grow ? mx : m_ref;
@@ -428,9 +455,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                 float p[8];
 #pragma unroll
                 for (int e = 0; e < 8; ++e) {
-                    p[e] = BIAS ? fa_ex2(sv[ch * 8 + e] - ref)
-                         : capped ? fa_ex2(fa_cap(sv[ch * 8 + e], k_in, k_out) - ref)
-                                  : fa_ex2(fmaf(sv[ch * 8 + e], scale_log2, -ref));
+                    p[e] = final_scores ? fa_ex2(sv[ch * 8 + e] - ref) : fa_ex2(fmaf(sv[ch * 8 + e], scale_log2, -ref));
                     ps4[e & 3] += p[e];
                 }
                 uint4 pk;
