@@ -429,15 +429,18 @@ mlstm_chain_kernel(float* __restrict__ part, float* __restrict__ part_n, const f
             for (int d = tid; d < D; d += 128) {
                 float* np_ = nvec + sh * D + d;
                 if (!ZLM_CHK(np_, 4)) continue;
-                float n = *np_;
+                float n = *np_, own[ML_CHAIN];
+#pragma unroll
+                for (int j = 0; j < ML_CHAIN; ++j) {
+                    const float* q = part_n + (at0 + (size_t)(p0 + j) * H) * D + d;
+                    own[j] = (j < cnt && ZLM_CHK(q, 4)) ? *q : 0.f;
+                }
 #pragma unroll
                 for (int j = 0; j < ML_CHAIN; ++j) {
                     if (j >= cnt) break;
                     float* q = part_n + (at0 + (size_t)(p0 + j) * H) * D + d;
-                    if (!ZLM_CHK(q, 4)) continue;
-                    const float own = *q;
-                    *q = n;
-                    n = fmaf(coef[j].x, n, coef[j].y * own);
+                    if (ZLM_CHK(q, 4)) *q = n;
+                    n = fmaf(coef[j].x, n, coef[j].y * own[j]);
                 }
                 *np_ = n;
             }
